@@ -19,14 +19,16 @@ from typing import Optional, Tuple
 
 @dataclass(frozen=True)
 class NormSpec:
-    """Root-mean-square norm over ``dim`` with a learned scale: x / sqrt(mean(x^2) + eps) * (offset + w).
-    ``offset`` is 0 where the scale is stored as it is applied and 1 where it is stored around zero;
+    """Root-mean-square norm over ``dim`` with a learned scale: x / sqrt(mean(x^2) + eps) * (offset + w) * gain.
+    ``offset`` is 0 where the scale is stored as it is applied and 1 where it is stored around zero; ``gain`` is a
+    constant of the design (the norm before a head whose logits are scaled carries that scale: the head is linear);
     ``suffix`` is what follows the part's prefix in the tensor's name."""
     dim: int
     eps: float
     kind: str = "rmsnorm"
     offset: float = 0.0
     suffix: str = ".weight"
+    gain: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -184,7 +186,8 @@ class LatentAttentionSpec:
     plain key is W_uk,h c and its value W_uv,h c; the score is (q_plain . k_plain + q_rot . k_rot) * scale.
     Only c and the rotated key part are cached; a layer that reads another layer's cache has no W_dkv.  ``sink``: a
     learned number per head joins the denominator.  ``head_gate``: head h's output is multiplied by
-    sigmoid((W_gate x)_h)."""
+    sigmoid((W_gate x)_h).  ``element_gate``: the concatenated heads are multiplied element by element by
+    sigmoid(W_gate x) instead.  ``window``: position i sees j with 0 <= i - j < window."""
     hidden_size: int
     num_heads: int
     head_dim: int
@@ -198,6 +201,7 @@ class LatentAttentionSpec:
     sink: bool = False
     window: Optional[int] = None
     head_gate: bool = False
+    element_gate: bool = False
     q_name: str = "q"
     gate_name: str = "g"
     dq_name: str = "dq"
@@ -430,8 +434,11 @@ class ClampedGluSpec:
 @dataclass(frozen=True)
 class RoutedExpertsSpec:
     """A mixture of ``n_experts`` feed-forwards of ``expert_size``, ``top_k`` per token: gated, down(silu(gate(x)) *
-    up(x)), or, with ``activation`` "relu2", plain, down(relu(up(x))^2).  The router's scores are in 32-bit
-    sigmoid(W_router x), or with ``scoring`` "softmax" the softmax of W_router x over all experts.  Experts form ``n_groups`` equal runs of neighbours; a group's
+    up(x)), or, with ``activation`` "relu2", plain, down(relu(up(x))^2), or, with "clamped_glu", gated by the unit of
+    ``ClampedGluSpec`` with ``limit`` (the shared expert: ``shared_limit``) and ``alpha``.  The router's logits are in
+    32-bit W_router x, plus a learned number per expert with ``router_bias_name``.  Its scores are their sigmoids, or
+    with ``scoring`` "softmax" their softmax over all experts, or with "softmax_chosen" the logits themselves for the
+    choice and, for the weights, the softmax over the chosen experts' logits alone.  Experts form ``n_groups`` equal runs of neighbours; a group's
     score is the sum of its ``group_score_top`` largest scores, and only experts of the ``keep_groups`` best
     groups can be chosen.  The chosen experts' outputs are added up weighted by their scores
     (``renormalize``: divided by the scores' sum plus ``renormalize_eps`` first), times ``weight_scale``.  With
@@ -452,9 +459,13 @@ class RoutedExpertsSpec:
     weight_scale: float = 1.0
     scoring: str = "sigmoid"
     activation: str = "silu_gated"
+    limit: float = 0.0
+    shared_limit: float = 0.0
+    alpha: float = 1.702
     shared_size: Optional[int] = None
     shared_prefix: str = "shared"
     correction_name: Optional[str] = None
+    router_bias_name: Optional[str] = None
     router_name: str = "router"
     expert_prefix: str = "e"
     gate_name: str = "gate"
@@ -553,11 +564,14 @@ class LayerCall:
     its weights are shared).  ``cache`` names the cache this call uses; by
     default every call has a cache of its own, numbered by its place in the
     order.  A call with ``writes_cache=False`` reads the cache of the earlier
-    call that owns it and stores nothing.
+    call that owns it and stores nothing.  With ``adds_embedding`` the embedding's
+    output (the residual stream as the first block of the model met it) is added
+    to the residual stream right before the block runs.
     """
     block: int
     cache: Optional[int] = None
     writes_cache: bool = True
+    adds_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -601,5 +615,16 @@ class ModelSpec:
             else:
                 if not (0 <= cache < n and out[cache].writes_cache):
                     raise ValueError(f"order[{n}] reads cache {cache}, which no earlier call owns")
-            out.append(LayerCall(call.block, cache, call.writes_cache))
+            out.append(LayerCall(call.block, cache, call.writes_cache, call.adds_embedding))
         return tuple(out)
+
+
+def looped_order(n_blocks: int, start: int, stop: int, times: int) -> Tuple[LayerCall, ...]:
+    """Blocks 0 .. start - 1, then start .. stop - 1 ``times`` times in a row with the same weights, then the rest; every
+    pass has caches of its own, and the embedding's output joins the stream before every pass but the first."""
+    if not 0 <= start < stop <= n_blocks or times < 1:
+        raise ValueError(f"blocks {start} .. {stop - 1} of {n_blocks}, {times} times, are no loop")
+    runs = [LayerCall(i) for i in range(start)]
+    for turn in range(times):
+        runs += [LayerCall(i, adds_embedding=turn > 0 and i == start) for i in range(start, stop)]
+    return tuple(runs + [LayerCall(i) for i in range(stop, n_blocks)])

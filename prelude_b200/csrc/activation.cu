@@ -296,3 +296,44 @@ PB_API int pb_relu2_(void* x, int dtype, long long n, cudaStream_t stream) {
     PB_CHECK_LAUNCH("relu2");
     return 0;
 }
+
+// A gate per element, in place: y[t, i] *= sigmoid(gate[t, i]) for columns of two row-major arrays, float32, one rounding.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* __restrict__ y, long long ldy, const T* __restrict__ gate, long long ldg, int cols) {
+    pb_grid_dep_launch();
+    pb_grid_dep_wait();
+    const size_t t = blockIdx.x;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    if (c >= cols) return;
+    T* yr = y + t * ldy + c;
+    const T* gr = gate + t * ldg + c;
+    __align__(16) T v[V], g[V];
+    if constexpr (V > 1) {
+        *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(yr);
+        *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gr);
+    } else {
+        v[0] = yr[0];
+        g[0] = gr[0];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) pb_st(v + e, pb_ld(v + e) / (1.0f + expf(-pb_ld(g + e))));
+    if constexpr (V > 1) *reinterpret_cast<uint4*>(yr) = *reinterpret_cast<const uint4*>(v);
+    else yr[0] = v[0];
+}
+
+PB_API int pb_sigmoid_gate_(void* y, long long ldy, const void* gate, long long ldg, int dtype, int n_tokens, int cols, cudaStream_t stream) {
+    PB_REQUIRE(n_tokens >= 0 && cols > 0 && ldy >= cols && ldg >= cols && y && gate, "sigmoid_gate: bad arguments T=%d cols=%d", n_tokens, cols);
+    if (n_tokens == 0) return 0;
+    const int v = dtype == PB_BF16 ? 8 : 4;
+    const bool vec = cols % v == 0 && ldy % v == 0 && ldg % v == 0 && pb_aligned(y, 16) && pb_aligned(gate, 16);
+    const int pieces = vec ? cols / v : cols;
+    PB_REQUIRE((pieces + 255) / 256 < 65536, "sigmoid_gate: rows of %d", cols);
+    const dim3 grid(n_tokens, (pieces + 255) / 256);
+    if (vec) {
+        PB_DISPATCH_DTYPE(dtype, T, (pb_launch(sigmoid_gate_kernel<T, 16 / (int)sizeof(T)>, grid, dim3(256), 0, stream, (T*)y, ldy, (const T*)gate, ldg, cols)));
+    } else {
+        PB_DISPATCH_DTYPE(dtype, T, (pb_launch(sigmoid_gate_kernel<T, 1>, grid, dim3(256), 0, stream, (T*)y, ldy, (const T*)gate, ldg, cols)));
+    }
+    PB_CHECK_LAUNCH("sigmoid_gate");
+    return 0;
+}

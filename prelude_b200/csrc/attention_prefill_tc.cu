@@ -65,6 +65,7 @@ struct PtParams {
     const float* sink;              // [n_heads] or null: exp(sink) joins the denominator
     const __nv_bfloat16* gate;      // [n_tokens, n_heads] rows ld_gate apart, or null: sigmoid(gate) multiplies the head's output
     long long ld_gate;
+    int gate_full;                  // the gate has an element for every element of the output: [n_tokens, n_heads * vd]
     int vd;                         // elements of a value row (at most 64 * VH)
     int flat;                       // keys and values lie in rows of their own maps (4 dimensions: element, row, head, page)
 };
@@ -398,9 +399,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 const int head = kvh * G + hg;
                 if (pp.sink != nullptr && m_ref != -INFINITY) l += ex2_approx(fmaf(pp.sink[head], 1.4426950408889634f, -m_ref));
                 float inv = l > 0.f ? 1.0f / l : 0.f;
-                if (pp.gate != nullptr && valid)
+                if (pp.gate != nullptr && valid && !pp.gate_full)
                     inv *= 1.0f / (1.0f + __expf(-__bfloat162float(pp.gate[(size_t)(q_base + tok0 + tl) * pp.ld_gate + head])));
                 __nv_bfloat16* dst = p.out + ((size_t)(q_base + tok0 + (valid ? tl : 0)) * p.n_heads + kvh * G + hg) * pp.vd;
+                const __nv_bfloat16* gates = pp.gate_full ? pp.gate + (size_t)(q_base + tok0 + (valid ? tl : 0)) * pp.ld_gate + (size_t)head * pp.vd : nullptr;
 #pragma unroll 1
                 for (int c = 0; c < T::VD; c += 32) {
                     uint32_t orr[32];
@@ -411,6 +413,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                         for (int i = 0; i < 32; i += 8) {
                             if (c + i >= pp.vd) break;
                             uint4 w;
+                            if (gates != nullptr) {
+                                const uint4 raw = *reinterpret_cast<const uint4*>(gates + c + i);
+                                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                                for (int u = 0; u < 4; ++u) {
+                                    const float2 g = __bfloat1622float2(h[u]);
+                                    orr[i + 2 * u] = __float_as_uint(__uint_as_float(orr[i + 2 * u]) / (1.0f + __expf(-g.x)));
+                                    orr[i + 2 * u + 1] = __float_as_uint(__uint_as_float(orr[i + 2 * u + 1]) / (1.0f + __expf(-g.y)));
+                                }
+                            }
                             w.x = pack_bf16(__uint_as_float(orr[i]) * inv, __uint_as_float(orr[i + 1]) * inv);
                             w.y = pack_bf16(__uint_as_float(orr[i + 2]) * inv, __uint_as_float(orr[i + 3]) * inv);
                             w.z = pack_bf16(__uint_as_float(orr[i + 4]) * inv, __uint_as_float(orr[i + 5]) * inv);
@@ -577,13 +589,15 @@ PB_API int pb_attention_prefill_tc_rows_supported(int kd, int vd) {
 // The same attention over keys and values of every query head's own, not in pages but in dense rows: kv [n_rows, n_heads,
 // kd + vd], a head's key before its value; a request's rows follow one another from a row that is a multiple of 128, and
 // row_blocks [requests, table_stride] lists its blocks of 128 rows (as a block table does pages).  q [n_tokens, n_heads, kd],
-// out [n_tokens, n_heads, vd].  Rows behind a request's last key must be finite (zeros).  Causal, no window; sink and gate as
-// for the masked entry point; tiles: 256 tokens each.
+// out [n_tokens, n_heads, vd].  Rows behind a request's last key, and rows of a listed block that no token of the step sees,
+// must be finite (zeros).  Causal; window as elsewhere (0: none), the blocks wholly before it need not be listed; sink and
+// gate as for the masked entry point, or, gate_full, a gate [n_tokens, n_heads * vd] that multiplies the output element by
+// element; tiles: 256 tokens each.
 PB_API int pb_attention_prefill_tc_rows_bf16(const void* q, const void* kv, void* out, const int32_t* row_blocks, int table_stride, int n_blocks,
                                              const int32_t* positions, const int32_t* token_seq, const int32_t* cu_q, const int32_t* q_start,
                                              const int32_t* tile_seq, const int32_t* tile_tok0, int n_tiles, int n_tokens, int n_heads, int kd,
-                                             int vd, float scale, const float* sink, const void* gate, long long ld_gate, int* status,
-                                             cudaStream_t stream) {
+                                             int vd, float scale, int window, const float* sink, const void* gate, long long ld_gate, int gate_full,
+                                             int* status, cudaStream_t stream) {
     PB_REQUIRE(pb_attention_prefill_tc_rows_supported(kd, vd), "attention_prefill_tc (rows): keys of %d, values of %d elements not taken", kd, vd);
     PtParams pp{};
     AttnParams& p = pp.a;
@@ -591,14 +605,17 @@ PB_API int pb_attention_prefill_tc_rows_bf16(const void* q, const void* kv, void
     p.out = (__nv_bfloat16*)out; p.block_table = row_blocks; p.positions = positions; p.token_seq = token_seq;
     p.cu_q = cu_q; p.q_start = q_start; p.tile_seq = tile_seq; p.tile_tok0 = tile_tok0; p.n_splits = 1;
     p.table_stride = table_stride; p.page_size = PT_KEYS; p.num_pages = n_blocks; p.n_tokens = n_tokens;
-    p.n_heads = n_heads; p.n_kv_heads = n_heads; p.head_dim = kd; p.window = 0; p.group = 1;
+    p.n_heads = n_heads; p.n_kv_heads = n_heads; p.head_dim = kd; p.window = window; p.group = 1;
     p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.swizzle = 0;
     if (int e = attn_check_common("attention_prefill_tc (rows)", p)) return e;
-    PB_REQUIRE(scale > 0.f && pb_aligned(out, 16) && (gate == nullptr || ld_gate >= n_heads), "attention_prefill_tc (rows): scale=%g, alignment or gate rows", (double)scale);
+    PB_REQUIRE(scale > 0.f && window >= 0 && pb_aligned(out, 16) && (gate == nullptr || ld_gate >= (gate_full ? (long long)n_heads * vd : n_heads)),
+               "attention_prefill_tc (rows): scale=%g, alignment or gate rows", (double)scale);
+    PB_REQUIRE(gate == nullptr || !gate_full || (pb_aligned(gate, 16) && ld_gate % 8 == 0), "attention_prefill_tc (rows): unaligned gate rows");
     PB_REQUIRE(n_tiles >= 0 && (long long)n_tiles * n_heads < (1ll << 31) && n_blocks > 0, "attention_prefill_tc (rows): bad grid");
     if (n_tiles == 0 || n_tokens == 0) return 0;
     pp.tok = 256; pp.q_rows = 128; pp.kv_rows = PT_KEYS; pp.flat = 1; pp.vd = vd;
     pp.sink = sink; pp.gate = (const __nv_bfloat16*)gate; pp.ld_gate = ld_gate;
+    pp.gate_full = gate != nullptr && gate_full ? 1 : 0;
     if (int e = get_encode()) return e;
     CUtensorMap mq, mk, mv;
     {

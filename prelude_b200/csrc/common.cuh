@@ -63,6 +63,11 @@ __device__ __forceinline__ float pb_gelu_tanh(float z) {
 }
 // a squashing in a norm's place: tanh(slope * v) * gain + shift, in float32
 __device__ __forceinline__ float pb_squash(float v, float slope, float gain, float shift) { return fmaf(tanhf(slope * v), gain, shift); }
+// the unit of PB_ACT_CLAMPED, in float32
+__device__ __forceinline__ float pb_clamped_unit(float g, float u, float limit, float alpha) {
+    const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
+    return a / (1.0f + expf(-alpha * a)) * (b + 1.0f);
+}
 __device__ __forceinline__ float pb_relu2(float v) { v = fmaxf(v, 0.f); return v * v; }
 __device__ __forceinline__ float pb_warp_max(float v) {
 #pragma unroll

@@ -605,21 +605,23 @@ PB_API int pb_gemm_pair_act_bf16(const void* A, const void* B, void* out, int ro
 // expert_rows_b, K] the experts' matrices one below the other; the device-side map (tile_expert, tile_row0 over
 // max_m_tiles row tiles of 256, offsets) says which rows are whose.  out [places, N] bfloat16 with N = expert_rows_b,
 // or, gated, N = expert_rows_b / 2 and silu(gate sums) * up sums (an expert's matrix: N gate rows, then N up rows); act:
-// PbAct (plain: PB_ACT_NONE or PB_ACT_RELU2).
+// PbAct (plain: PB_ACT_NONE or PB_ACT_RELU2; gated: PB_ACT_SILU, or PB_ACT_CLAMPED with limit and alpha).
 PB_API int pb_gemm_pair_grouped_bf16(const void* A, const void* B, void* out, int places, int expert_rows_b, int n_experts, int K,
-                                     long long lda, long long ldb, long long ldo, int gated, int act, const int32_t* tile_expert,
+                                     long long lda, long long ldb, long long ldo, int gated, int act, float limit, float alpha, const int32_t* tile_expert,
                                      const int32_t* tile_row0, const int32_t* offsets, int max_m_tiles, int max_pairs,
                                      int* status, cudaStream_t stream) {
     PB_REQUIRE(n_experts > 0 && max_m_tiles >= 0 && pb_gemm_pair_supported(places, expert_rows_b, K, lda, ldb, gated),
                "gemm_pair (grouped): places=%d rows per expert=%d K=%d lda=%lld ldb=%lld not taken", places, expert_rows_b, K, lda, ldb);
     PB_REQUIRE((long long)n_experts * expert_rows_b < (1ll << 31), "gemm_pair (grouped): too many rows of B");
     PB_REQUIRE(A && B && out && tile_expert && tile_row0 && offsets && pb_aligned(A, 16) && pb_aligned(B, 16), "gemm_pair (grouped): null or unaligned pointer");
+    PB_REQUIRE(gated ? act == PB_ACT_SILU || (act == PB_ACT_CLAMPED && limit > 0.f) : act == PB_ACT_NONE || act == PB_ACT_RELU2,
+               "gemm_pair (grouped): activation %d in the %s form, limit %g", act, gated ? "gated" : "plain", (double)limit);
     if (max_m_tiles == 0) return 0;
     if (int e = get_encode()) return e;
     GpParams p{};
     p.out = (__nv_bfloat16*)out; p.bias = nullptr; p.status = status; p.ldo = ldo;
     p.rows_a = places; p.rows_b = expert_rows_b; p.K = K; p.gated = gated ? 1 : 0; p.b_is_constant = 1;
-    p.act = act;
+    p.act = act; p.limit = limit; p.alpha = alpha;
     p.tile_expert = tile_expert; p.tile_row0 = tile_row0; p.offsets = offsets;
     p.expert_rows_b = expert_rows_b; p.map_rows_b = n_experts * expert_rows_b;
     p.out_cols = gated ? expert_rows_b / 2 : expert_rows_b;

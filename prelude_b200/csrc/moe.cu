@@ -3,7 +3,8 @@
 // counts, offsets and the map from tiles to experts stay on the device, so a step through a mixture of experts
 // has the shape of its token count alone and can be recorded.
 //
-//   route    scores s = sigmoid(z) of float32 router logits, or their softmax over all experts; experts form `groups` equal runs of neighbours, a
+//   route    scores s = sigmoid(z) of float32 router logits (plus a bias per expert where there is one), or their softmax over
+//            all experts, or z itself, the weights then being the softmax over the chosen experts' z alone; experts form `groups` equal runs of neighbours, a
 //            group's score is the sum of its `gtop` largest scores, only experts of the `keep` best groups can
 //            be chosen; the `top` largest allowed scores are chosen (ties: the smaller index), their weights are
 //            the scores themselves (or, with `renorm`, divided by their sum plus `renorm_eps`) times `scale`.  With a `correction` per expert the
@@ -12,13 +13,14 @@
 //   sort     slot i = token * top + choice.  The slots are grouped by expert: offsets[e] .. offsets[e + 1] are the
 //            places of expert e, order[place] = slot, place_of[slot] = place, and the places are cut into row
 //            tiles of MOE_BM that never span two experts (tile_expert, tile_row0; -1 behind the last tile).
-//   products h[place] = silu(Wg_e x) * (Wu_e x), or relu(Wu_e x)^2, with x the row of slot / top, then
+//   products h[place] = silu(Wg_e x) * (Wu_e x), or the clamped unit of the two, or relu(Wu_e x)^2, with x the row of slot / top, then
 //            y[place] = Wd_e h[place].
 //            An output element is summed over k in ascending order by one thread (float32 units) or one
 //            tensor-core accumulator (bfloat16), whatever its place in the tile, so a token's result does not
 //            depend on who else chose the expert.
 //   combine  out[t] = sum over choices c, in order, of w[t, c] * y[place_of[t * top + c]] (+ the output of an expert that
-//            every token runs), in float32; or the same added to the residual stream, with the squashing that follows.
+//            every token runs), in float32; or the same added to the residual stream, with the squashing that follows; or the
+//            same normed, added to the residual stream, and the sum normed.
 //
 // A decode step's few tokens take a shorter way: router logits and choice in one kernel (pb_moe_route_few), no sort (the
 // places are the slots themselves), and products that find an expert's rows by looking through the choices.
@@ -220,9 +222,12 @@ __device__ __forceinline__ void moe_warp_argmax(float& val, int& idx) {
     }
 }
 
+enum MoeScoring : int { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_SOFTMAX_CHOSEN = 2 };
+
 struct MoeRouteArgs {
     const float* correction;                                 // float32 [n_experts] or null
-    int n_experts, top, groups, keep, gtop, renorm, softmax;
+    const float* bias;                                       // float32 [n_experts], added to the logits, or null
+    int n_experts, top, groups, keep, gtop, renorm, scoring; // MoeScoring
     float renorm_eps, scale;
 };
 
@@ -233,17 +238,21 @@ __device__ __forceinline__ void moe_route_token(const float* z, const MoeRouteAr
     const int n_experts = a.n_experts, groups = a.groups, per = n_experts / groups;
     const float NONE = -INFINITY;                            // below every choice score, negative ones included
     float zmax = 0.f, inv_sum = 1.f;
-    if (a.softmax) {
+    auto logit = [&](int e) { return a.bias ? z[e] + a.bias[e] : z[e]; };
+    if (a.scoring == MOE_SOFTMAX) {
         float m = NONE;
 #pragma unroll
-        for (int i = 0; i < SLOTS; ++i) { const int e = lane + 32 * i; if (e < n_experts) m = fmaxf(m, z[e]); }
+        for (int i = 0; i < SLOTS; ++i) { const int e = lane + 32 * i; if (e < n_experts) m = fmaxf(m, logit(e)); }
         zmax = pb_warp_max(m);
         float sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < SLOTS; ++i) { const int e = lane + 32 * i; if (e < n_experts) sum += expf(z[e] - zmax); }
+        for (int i = 0; i < SLOTS; ++i) { const int e = lane + 32 * i; if (e < n_experts) sum += expf(logit(e) - zmax); }
         inv_sum = 1.0f / pb_warp_sum(sum);
     }
-    auto score = [&](int e) { return a.softmax ? expf(z[e] - zmax) * inv_sum : 1.0f / (1.0f + expf(-z[e])); };
+    auto score = [&](int e) {
+        const float v = logit(e);
+        return a.scoring == MOE_SOFTMAX ? expf(v - zmax) * inv_sum : a.scoring == MOE_SOFTMAX_CHOSEN ? v : 1.0f / (1.0f + expf(-v));
+    };
     float sc[SLOTS];                                         // what the choice goes by
 #pragma unroll
     for (int i = 0; i < SLOTS; ++i) {
@@ -303,6 +312,11 @@ __device__ __forceinline__ void moe_route_token(const float* z, const MoeRouteAr
         total += val;
         if (lane == r) { my_id = idx; my_w = val; }
     }
+    if (a.scoring == MOE_SOFTMAX_CHOSEN) {                   // of the chosen logits alone, whatever the order of the choice
+        const float top_z = pb_warp_max(lane < a.top ? my_w : NONE);
+        my_w = lane < a.top ? expf(my_w - top_z) : 0.f;
+        my_w /= pb_warp_sum(my_w);
+    }
     if (lane < a.top) {
         ids[lane] = my_id;
         weights[lane] = (a.renorm ? my_w / (total + a.renorm_eps) : my_w) * a.scale;
@@ -324,16 +338,19 @@ static int moe_route_check(int n_tokens, const MoeRouteArgs& a) {
                "moe_route: bad sizes T=%d E=%d top=%d", n_tokens, a.n_experts, a.top);
     PB_REQUIRE(a.groups > 0 && a.groups <= MOE_MAX_GROUPS && a.n_experts % a.groups == 0 && a.keep > 0 && a.keep <= a.groups && a.gtop > 0 &&
                a.gtop <= MOE_MAX_GTOP, "moe_route: %d groups, keep %d, group score over %d", a.groups, a.keep, a.gtop);
+    PB_REQUIRE(a.scoring == MOE_SIGMOID || a.scoring == MOE_SOFTMAX || (a.scoring == MOE_SOFTMAX_CHOSEN && !a.renorm),
+               "moe_route: scoring %d, renormalized %d", a.scoring, a.renorm);
     PB_REQUIRE(a.top <= a.keep * (a.n_experts / a.groups), "moe_route: top=%d experts cannot come from %d groups of %d", a.top, a.keep,
                a.n_experts / a.groups);
     return 0;
 }
 
-// correction: float32 [n_experts] added to the scores for the choice only, or null; softmax: scores are the softmax of the
-// logits (else their sigmoid); renorm: weights divided by their sum + renorm_eps; all weights times scale.
-PB_API int pb_moe_route(const float* logits, const float* correction, int n_tokens, int n_experts, int top, int groups, int keep,
-                        int gtop, int softmax, int renorm, float renorm_eps, float scale, int32_t* ids, float* weights, cudaStream_t stream) {
-    const MoeRouteArgs args{correction, n_experts, top, groups, keep, gtop, renorm, softmax, renorm_eps, scale};
+// correction: float32 [n_experts] added to the scores for the choice only, or null; bias: float32 [n_experts] added to the
+// logits, or null; scoring: MoeScoring; renorm: weights divided by their sum + renorm_eps (not with MOE_SOFTMAX_CHOSEN, whose
+// weights add up to one); all weights times scale.
+PB_API int pb_moe_route(const float* logits, const float* correction, const float* bias, int n_tokens, int n_experts, int top, int groups,
+                        int keep, int gtop, int scoring, int renorm, float renorm_eps, float scale, int32_t* ids, float* weights, cudaStream_t stream) {
+    const MoeRouteArgs args{correction, bias, n_experts, top, groups, keep, gtop, renorm, scoring, renorm_eps, scale};
     if (int e = moe_route_check(n_tokens, args)) return e;
     PB_REQUIRE(logits && ids && weights, "moe_route: null pointer");
     if (n_tokens == 0) return 0;
@@ -414,10 +431,10 @@ PB_API int pb_moe_route_few_supported(int n_experts, int K, int dtype) {
 }
 
 // x [n_tokens, K] with row stride ldx, W [n_experts, K], both of type dtype; the rest as pb_moe_route.
-PB_API int pb_moe_route_few(const void* x, long long ldx, const void* W, int dtype, int K, const float* correction, int n_tokens, int n_experts,
-                            int top, int groups, int keep, int gtop, int softmax, int renorm, float renorm_eps, float scale, int32_t* ids,
+PB_API int pb_moe_route_few(const void* x, long long ldx, const void* W, int dtype, int K, const float* correction, const float* bias,
+                            int n_tokens, int n_experts, int top, int groups, int keep, int gtop, int scoring, int renorm, float renorm_eps, float scale, int32_t* ids,
                             float* weights, cudaStream_t stream) {
-    const MoeRouteArgs args{correction, n_experts, top, groups, keep, gtop, renorm, softmax, renorm_eps, scale};
+    const MoeRouteArgs args{correction, bias, n_experts, top, groups, keep, gtop, renorm, scoring, renorm_eps, scale};
     if (int e = moe_route_check(n_tokens, args)) return e;
     PB_REQUIRE(pb_moe_route_few_supported(n_experts, K, dtype) && ldx >= K && ldx % (dtype == PB_BF16 ? 8 : 4) == 0,
                "moe_route_few: E=%d K=%d ldx=%lld not taken", n_experts, K, ldx);
@@ -509,12 +526,23 @@ PB_API int pb_moe_sort(const int32_t* ids, int n_slots, int n_experts, int32_t* 
 // expert's weight being [2 N, K], gate rows first.  src(place) = order[place] / a_div when `order` is given (the
 // token of a slot), else the place itself.
 // ---------------------------------------------------------------------------------------------------------------
+struct MoeAct {
+    int kind;                                                // PbAct: gated PB_ACT_SILU or PB_ACT_CLAMPED, plain PB_ACT_NONE or PB_ACT_RELU2
+    float limit, alpha;                                      // of the clamped unit
+};
+__device__ __forceinline__ float moe_gate(float g, float u, const MoeAct& a) {
+    return a.kind == PB_ACT_CLAMPED ? pb_clamped_unit(g, u, a.limit, a.alpha) : g / (1.0f + expf(-g)) * u;
+}
+static bool moe_act_ok(int gated, const MoeAct& a) {
+    return gated ? a.kind == PB_ACT_SILU || (a.kind == PB_ACT_CLAMPED && a.limit > 0.f) : a.kind == PB_ACT_NONE || a.kind == PB_ACT_RELU2;
+}
+
 template <typename T, typename TC, bool GATED>
 __global__ void __launch_bounds__(256) moe_gemm_fma_kernel(const T* __restrict__ A, long long lda, const int32_t* __restrict__ order,
                                                            int a_div, const T* __restrict__ W, long long w_expert_stride, int N,
                                                            int K, const int32_t* __restrict__ tile_expert,
                                                            const int32_t* __restrict__ tile_row0,
-                                                           const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, int act) {
+                                                           const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, MoeAct act) {
     pb_grid_dep_launch();
     pb_grid_dep_wait();
     const int e = tile_expert[blockIdx.x];
@@ -578,8 +606,8 @@ __global__ void __launch_bounds__(256) moe_gemm_fma_kernel(const T* __restrict__
             const int gn = n0 + tx * 4 + j;
             if (gn >= N) continue;
             float v = acc[0][i][j];
-            if (GATED) v = v / (1.0f + expf(-v)) * acc[GATED ? 1 : 0][i][j];
-            else if (act == PB_ACT_RELU2) v = pb_relu2(v);
+            if (GATED) v = moe_gate(v, acc[GATED ? 1 : 0][i][j], act);
+            else if (act.kind == PB_ACT_RELU2) v = pb_relu2(v);
             pb_st(C + (size_t)p * ldc + gn, v);
         }
     }
@@ -599,7 +627,7 @@ __global__ void __launch_bounds__(256) moe_gemm_bf16_kernel(const __nv_bfloat16*
                                                             const __nv_bfloat16* __restrict__ W, long long w_expert_stride, int N,
                                                             int K, const int32_t* __restrict__ tile_expert,
                                                             const int32_t* __restrict__ tile_row0,
-                                                            const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, int act) {
+                                                            const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, MoeAct act) {
     using namespace nvcuda;
     pb_grid_dep_launch();
     pb_grid_dep_wait();
@@ -656,10 +684,9 @@ __global__ void __launch_bounds__(256) moe_gemm_bf16_kernel(const __nv_bfloat16*
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int i = 0; i < acc[0][j].num_elements; ++i) {
-                const float v = acc[0][j].x[i];
-                acc[0][j].x[i] = v / (1.0f + expf(-v)) * acc[GATED ? 1 : 0][j].x[i];
+                acc[0][j].x[i] = moe_gate(acc[0][j].x[i], acc[GATED ? 1 : 0][j].x[i], act);
             }
-    } else if (act == PB_ACT_RELU2) {
+    } else if (act.kind == PB_ACT_RELU2) {
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -707,7 +734,7 @@ __global__ void __launch_bounds__(256) moe_gemm_large_kernel(const __nv_bfloat16
                                                              const __nv_bfloat16* __restrict__ W, long long w_expert_stride, int N,
                                                              int K, const int32_t* __restrict__ tile_expert,
                                                              const int32_t* __restrict__ tile_row0,
-                                                             const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, int act) {
+                                                             const int32_t* __restrict__ offsets, TC* __restrict__ C, long long ldc, MoeAct act) {
     pb_grid_dep_launch();
     pb_grid_dep_wait();
     const int e = tile_expert[blockIdx.x];
@@ -799,8 +826,8 @@ __global__ void __launch_bounds__(256) moe_gemm_large_kernel(const __nv_bfloat16
                     const int col = n0 + (GATED ? wn * 16 : wn * 32) + nt * 8 + 2 * t4 + q;
                     if (col >= N) continue;
                     float v = acc[mi][nt][2 * h + q];
-                    if (GATED) v = v / (1.0f + expf(-v)) * acc[mi][nt + (GATED ? 2 : 0)][2 * h + q];
-                    else if (act == PB_ACT_RELU2) v = pb_relu2(v);
+                    if (GATED) v = moe_gate(v, acc[mi][nt + (GATED ? 2 : 0)][2 * h + q], act);
+                    else if (act.kind == PB_ACT_RELU2) v = pb_relu2(v);
                     pb_st(crow + col, v);
                 }
             }
@@ -810,15 +837,17 @@ __global__ void __launch_bounds__(256) moe_gemm_large_kernel(const __nv_bfloat16
 
 // A [*, K] with row stride lda; order null or int32 [places]; W [E, (2) N, K] dense, w_expert_stride elements from one
 // expert to the next; C [places, N] with row stride ldc, of type out_dtype (float32 or the input's).  grid: max_tiles.
-// act: of the plain form, PB_ACT_NONE or PB_ACT_RELU2.
+// act, limit, alpha: see MoeAct.
 PB_API int pb_moe_gemm(const void* A, long long lda, const int32_t* order, int a_div, const void* W, long long w_expert_stride,
-                       int N, int K, int gated, int act, const int32_t* tile_expert, const int32_t* tile_row0, const int32_t* offsets,
+                       int N, int K, int gated, int act_kind, float limit, float alpha, const int32_t* tile_expert, const int32_t* tile_row0, const int32_t* offsets,
                        int max_tiles, int tile_rows, void* C, long long ldc, int dtype, int out_dtype, cudaStream_t stream) {
     PB_REQUIRE(tile_rows == MOE_BM || tile_rows == MOE_BM_LARGE, "moe_gemm: tiles have %d or %d rows", MOE_BM, MOE_BM_LARGE);
     PB_REQUIRE(N > 0 && K > 0 && max_tiles >= 0 && a_div > 0, "moe_gemm: bad sizes N=%d K=%d", N, K);
     PB_REQUIRE(lda >= K && ldc >= N && w_expert_stride >= (long long)(gated ? 2 : 1) * N * K, "moe_gemm: a stride is shorter than its row");
     PB_REQUIRE(A && W && C && tile_expert && tile_row0 && offsets, "moe_gemm: null pointer");
     PB_REQUIRE(out_dtype == PB_F32 || out_dtype == dtype, "moe_gemm: output is float32 or of the input's type");
+    const MoeAct act{act_kind, limit, alpha};
+    PB_REQUIRE(moe_act_ok(gated, act), "moe_gemm: activation %d in the %s form, limit %g", act_kind, gated ? "gated" : "plain", (double)limit);
     if (max_tiles == 0) return 0;
     dim3 grid(max_tiles, (N + MOE_BN - 1) / MOE_BN);
     PB_REQUIRE(grid.y < 65536, "moe_gemm: N=%d too large", N);
@@ -897,7 +926,7 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const __nv_bfloat16* __re
                                                        const __nv_bfloat16* __restrict__ W, long long w_expert_stride, int N, int K,
                                                        const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ tile_row0,
                                                        const int32_t* __restrict__ offsets, const int32_t* __restrict__ ids, int n_slots,
-                                                       TC* __restrict__ C, long long ldc, int act) {
+                                                       TC* __restrict__ C, long long ldc, MoeAct act) {
     __shared__ int slots_s[MOE_GEMV_SLOTS];
     __shared__ int count_s;
     pb_grid_dep_launch();
@@ -981,8 +1010,8 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const __nv_bfloat16* __re
             for (int q = 0; q < NF; ++q)
                 if (lane == NF * r + q && r0 + r < rows && f0 + q < N) {
                     float v = acc[q][r];
-                    if (GATED) v = v / (1.0f + expf(-v)) * acc[GATED ? 2 + q : q][r];
-                    else if (act == PB_ACT_RELU2) v = pb_relu2(v);
+                    if (GATED) v = moe_gate(v, acc[GATED ? 2 + q : q][r], act);
+                    else if (act.kind == PB_ACT_RELU2) v = pb_relu2(v);
                     pb_st(C + (size_t)place[r] * ldc + f0 + q, v);
                 }
     };
@@ -998,13 +1027,15 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const __nv_bfloat16* __re
 // max_tiles = the number of experts) the map, order and offsets are not needed: rows of A are slot / a_div (a_div 1: the
 // slot's own row), rows of C the slots.
 PB_API int pb_moe_gemv(const void* A, long long lda, const int32_t* order, int a_div, const void* W, long long w_expert_stride,
-                       int N, int K, int gated, int act, const int32_t* tile_expert, const int32_t* tile_row0, const int32_t* offsets,
-                       int max_tiles, const int32_t* ids, int n_slots, void* C, long long ldc, int out_dtype, cudaStream_t stream) {
+                       int N, int K, int gated, int act_kind, float limit, float alpha, const int32_t* tile_expert, const int32_t* tile_row0,
+                       const int32_t* offsets, int max_tiles, const int32_t* ids, int n_slots, void* C, long long ldc, int out_dtype, cudaStream_t stream) {
     PB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && lda % 8 == 0 && w_expert_stride % 8 == 0 && max_tiles >= 0 && a_div > 0,
                "moe_gemv: N=%d K=%d lda=%lld: K and the strides in multiples of 8", N, K, lda);
     PB_REQUIRE(A && W && C && pb_aligned(A, 16) && pb_aligned(W, 16), "moe_gemv: null or unaligned pointer");
     PB_REQUIRE(ids ? (n_slots >= 0 && n_slots <= MOE_GEMV_SLOTS) : (tile_expert && tile_row0 && offsets), "moe_gemv: neither a map nor a list of choices (%d)", n_slots);
     PB_REQUIRE(lda >= K && ldc >= N && w_expert_stride >= (long long)(gated ? 2 : 1) * N * K, "moe_gemv: a stride is shorter than its row");
+    const MoeAct act{act_kind, limit, alpha};
+    PB_REQUIRE(moe_act_ok(gated, act), "moe_gemv: activation %d in the %s form, limit %g", act_kind, gated ? "gated" : "plain", (double)limit);
     if (max_tiles == 0 || (ids && n_slots == 0)) return 0;
     const int per_block = gated ? 16 : 32;
     dim3 grid(max_tiles, (N + per_block - 1) / per_block);
@@ -1230,5 +1261,176 @@ PB_API int pb_moe_sum(const void* y, int y_dtype, const int32_t* place_of, const
     }
 #undef MOE_SUM
     PB_CHECK_LAUNCH("moe_sum");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// The weighted sum where the sublayer's output is normed before it joins the residual stream, with that norm, the add and
+// the norm that follows:
+//   v[t] = sum_c w[t, c] * y[place(t, c), :] + shared[t, :]
+//   res[t] += v / sqrt(mean(v^2) + eps_v) * gain_v (+ plus[t]) ;  out[t] = res / sqrt(mean(res^2) + eps) * gain
+// One block a token, the row in registers between the passes, float32 throughout; v is rounded nowhere.  The block's size
+// depends on the row's width alone.  With `rows` row i of out is made from token rows[i], and res is left alone.
+// ---------------------------------------------------------------------------------------------------------------
+struct MoeSumNormArgs {
+    const int32_t* place_of;
+    const float* weights;
+    int shared_parts;
+    size_t shared_stride;
+    const float* gain_v;
+    const float* gain;
+    const float* plus;
+    float* res;
+    const int32_t* rows;
+    float eps_v, eps;
+    int n_tokens, top, width;
+};
+
+__device__ __forceinline__ float moe_block_sum(float v, float* red) {
+    v = pb_warp_sum(v);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    float total = 0.f;
+    for (int i = 0; i < nwarp; ++i) total += red[i];         // the same order in every thread
+    return total;
+}
+
+template <typename TY, typename TS, typename TO, int V, int IT>
+__global__ void __launch_bounds__(256) moe_sum_normed_kernel(const TY* __restrict__ y, const TS* __restrict__ shared, TO* __restrict__ out, MoeSumNormArgs a) {
+    pb_grid_dep_launch();
+    __shared__ float red[2][8];
+    const int i = blockIdx.x;
+    float gv[IT][V], g[IT][V];
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {                        // written by no kernel: before the wait
+        const int col = (it * blockDim.x + threadIdx.x) * V;
+        if (col < a.width) { moe_ldv<V>(a.gain_v + col, gv[it]); moe_ldv<V>(a.gain + col, g[it]); }
+    }
+    pb_grid_dep_wait();
+    const int t = a.rows ? a.rows[i] : i;
+    if (t < 0 || t >= a.n_tokens) {                          // the whole block
+#pragma unroll
+        for (int it = 0; it < IT; ++it) {
+            const int col = (it * blockDim.x + threadIdx.x) * V;
+            float zero[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) zero[e] = 0.f;
+            if (col < a.width) moe_stv<V>(out + (size_t)i * a.width + col, zero);
+        }
+        return;
+    }
+    float v[IT][V], r[IT][V];
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int col = (it * blockDim.x + threadIdx.x) * V;
+        if (col >= a.width) continue;
+        moe_ldv<V>(a.res + (size_t)t * a.width + col, r[it]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[it][e] = 0.f;
+        for (int c0 = 0; c0 < a.top; c0 += 4) {              // four choices' loads in flight
+            float yv[4][V], w[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                if (c0 + u < a.top) {
+                    const int slot = t * a.top + c0 + u;
+                    w[u] = a.weights[slot];
+                    moe_ldv<V>(y + (size_t)(a.place_of ? a.place_of[slot] : slot) * a.width + col, yv[u]);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                if (c0 + u < a.top) {
+#pragma unroll
+                    for (int e = 0; e < V; ++e) v[it][e] = fmaf(w[u], yv[u][e], v[it][e]);
+                }
+        }
+        for (int p = 0; p < a.shared_parts; ++p) {
+            float sv[V];
+            moe_ldv<V>(shared + (size_t)p * a.shared_stride + (size_t)t * a.width + col, sv);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[it][e] += sv[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += v[it][e] * v[it][e];
+    }
+    const float inv_v = 1.0f / sqrtf(moe_block_sum(ss, red[0]) / (float)a.width + a.eps_v);
+    ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int col = (it * blockDim.x + threadIdx.x) * V;
+        if (col >= a.width) continue;
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[it][e] += v[it][e] * inv_v * gv[it][e];
+        if (a.plus) {
+            float pv[V];
+            moe_ldv<V>(a.plus + (size_t)t * a.width + col, pv);
+#pragma unroll
+            for (int e = 0; e < V; ++e) r[it][e] += pv[e];
+        }
+        if (a.rows == nullptr) moe_stv<V>(a.res + (size_t)t * a.width + col, r[it]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += r[it][e] * r[it][e];
+    }
+    const float inv = 1.0f / sqrtf(moe_block_sum(ss, red[1]) / (float)a.width + a.eps);
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int col = (it * blockDim.x + threadIdx.x) * V;
+        if (col >= a.width) continue;
+        float o[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = r[it][e] * inv * g[it][e];
+        moe_stv<V>(out + (size_t)i * a.width + col, o);
+    }
+}
+
+// Whether pb_moe_sum_normed takes rows of `width`: multiples of the elements of 16 bytes, what a block's registers hold.
+PB_API int pb_moe_sum_normed_supported(int width, int dtype) {
+    const int v = dtype == PB_F32 ? 4 : 8;
+    return width > 0 && width % v == 0 && width / v <= 256 * (dtype == PB_F32 ? 8 : 4) ? 1 : 0;
+}
+
+// y, shared as for pb_moe_sum; gain_v, gain float32 [width] as applied; res float32 [n_tokens, width]; plus null or of res's
+// shape (without rows); rows null or int32 [n_out]; out [n_out, width] of type dtype.
+PB_API int pb_moe_sum_normed(const void* y, int y_dtype, const int32_t* place_of, const float* weights, const void* shared, int shared_dtype,
+                             int shared_parts, long long shared_stride, const float* gain_v, float eps_v, float* res, const float* plus,
+                             const int32_t* rows, const float* gain, float eps, void* out, int dtype, int n_out, int n_tokens, int top, int width,
+                             cudaStream_t stream) {
+    PB_REQUIRE((y_dtype == PB_F32 || y_dtype == dtype) && (shared_parts == 0 || shared_dtype == PB_F32 || shared_dtype == dtype),
+               "moe_sum_normed: operands are float32 or of the output's type");
+    PB_REQUIRE(n_out >= 0 && n_tokens >= 0 && top > 0 && shared_parts >= 0 && shared_parts <= 64 && pb_moe_sum_normed_supported(width, dtype),
+               "moe_sum_normed: bad sizes, rows of %d", width);
+    PB_REQUIRE(y && weights && out && res && gain_v && gain && (shared_parts == 0 || shared), "moe_sum_normed: null pointer");
+    PB_REQUIRE(rows != nullptr ? plus == nullptr : n_out == n_tokens, "moe_sum_normed: rows and outputs do not fit");
+    const int V = dtype == PB_F32 ? 4 : 8;
+    PB_REQUIRE(pb_aligned(y, 16) && pb_aligned(out, 16) && pb_aligned(res, 16) && pb_aligned(gain, 16) && pb_aligned(gain_v, 16) && pb_aligned(plus, 16) &&
+               (shared_parts == 0 || (pb_aligned(shared, 16) && shared_stride % V == 0)), "moe_sum_normed: unaligned pointer");
+    if (n_out == 0) return 0;
+    const int pieces = width / V;
+    int threads = 32;
+    while (threads < 256 && threads < pieces) threads <<= 1;
+    const int its = (pieces + threads - 1) / threads;
+    const MoeSumNormArgs a{place_of, weights, shared_parts, (size_t)shared_stride, gain_v, gain, plus, res, rows, eps_v, eps, n_tokens, top, width};
+#define MOE_SUM_AT(TY, TS, TO, VV, IT) \
+    pb_launch(moe_sum_normed_kernel<TY, TS, TO, VV, IT>, dim3(n_out), dim3(threads), 0, stream, (const TY*)y, (const TS*)shared, (TO*)out, a)
+#define MOE_SUM(TY, TS, TO, VV)                                  \
+    do {                                                         \
+        if (its <= 1) MOE_SUM_AT(TY, TS, TO, VV, 1);             \
+        else if (its <= 2) MOE_SUM_AT(TY, TS, TO, VV, 2);        \
+        else if (its <= 4) MOE_SUM_AT(TY, TS, TO, VV, 4);        \
+        else MOE_SUM_AT(TY, TS, TO, VV, 8);                      \
+    } while (0)
+    if (dtype == PB_F32) MOE_SUM(float, float, float, 4);
+    else if (dtype == PB_BF16) {
+        const bool sf = shared_parts == 0 || shared_dtype == PB_F32;
+        if (y_dtype == PB_F32) { if (sf) MOE_SUM(float, float, __nv_bfloat16, 8); else MOE_SUM(float, __nv_bfloat16, __nv_bfloat16, 8); }
+        else { if (sf) MOE_SUM(__nv_bfloat16, float, __nv_bfloat16, 8); else MOE_SUM(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16, 8); }
+    } else {
+        return pb_fail("moe_sum_normed: unknown element type code %d", dtype);
+    }
+#undef MOE_SUM
+#undef MOE_SUM_AT
+    PB_CHECK_LAUNCH("moe_sum_normed");
     return 0;
 }

@@ -325,14 +325,14 @@ PB_API int pb_rmsnorm(const void* x, const float* w, void* y, int dtype, int row
 }
 
 // A sublayer's output that is normed before it joins the residual stream, fused with the norm that follows:
-//   res += x / sqrt(mean(x^2) + eps_x) * wx ;  y = res / sqrt(mean(res^2) + eps) * w
+//   res += x / sqrt(mean(x^2) + eps_x) * wx (+ plus) ;  y = res / sqrt(mean(res^2) + eps) * w
 // one block per row, all in float32; x is rounded nowhere between its norm and the sum.  Without w and y only the
-// sum is made.  With `rows` (the gather form) row i of y is made from row rows[i] of x and res, and res is left alone.
+// sum is made.  plus: null, or what also joins the stream there (a loop of layers takes the embedding's output again).  With `rows` (the gather form) row i of y is made from row rows[i] of x and res, and res is left alone.
 // The row is kept in shared memory between the passes where it fits, else it is read again.
 template <typename TX, typename TY>
 __global__ void normed_add_rmsnorm_kernel(const TX* __restrict__ x, const float* __restrict__ wx, float eps_x,
-                                          float* __restrict__ res, const int32_t* __restrict__ rows, int n_rows_total,
-                                          const float* __restrict__ w, TY* __restrict__ y, int width, float eps, int keep) {
+                                          float* __restrict__ res, const float* __restrict__ plus, const int32_t* __restrict__ rows,
+                                          int n_rows_total, const float* __restrict__ w, TY* __restrict__ y, int width, float eps, int keep) {
     pb_grid_dep_launch();
     pb_grid_dep_wait();
     extern __shared__ float row_s[];
@@ -355,6 +355,7 @@ __global__ void normed_add_rmsnorm_kernel(const TX* __restrict__ x, const float*
     ss = 0.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         float v = r[i] + (keep ? row_s[i] : pb_ld(xr + i)) * inv_x * wx[i];
+        if (plus) v += plus[(size_t)src * width + i];
         if (rows == nullptr) r[i] = v;
         if (keep) row_s[i] = v;
         ss += v * v;
@@ -373,8 +374,8 @@ __global__ void normed_add_rmsnorm_kernel(const TX* __restrict__ x, const float*
 // stored.  width % 4 == 0, width <= 4 * blockDim * ITERS.
 template <typename TX, typename TY, int ITERS>
 __global__ void normed_add_rmsnorm_vec4_kernel(const TX* __restrict__ x, const float* __restrict__ wx, float eps_x,
-                                               float* __restrict__ res, const int32_t* __restrict__ rows, int n_rows_total,
-                                               const float* __restrict__ w, TY* __restrict__ y, int width, float eps) {
+                                               float* __restrict__ res, const float* __restrict__ plus, const int32_t* __restrict__ rows,
+                                               int n_rows_total, const float* __restrict__ w, TY* __restrict__ y, int width, float eps) {
     pb_grid_dep_launch();
     __shared__ float red[32];
     const int n4 = width >> 2;
@@ -426,6 +427,10 @@ __global__ void normed_add_rmsnorm_vec4_kernel(const TX* __restrict__ x, const f
             float4 v = rv[it];
             v.x += xv[it].x * inv_x * gx[it].x; v.y += xv[it].y * inv_x * gx[it].y;
             v.z += xv[it].z * inv_x * gx[it].z; v.w += xv[it].w * inv_x * gx[it].w;
+            if (plus != nullptr) {
+                const float4 e = reinterpret_cast<const float4*>(plus + row * width)[i];
+                v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+            }
             if (rows == nullptr) reinterpret_cast<float4*>(res + row * width)[i] = v;
             rv[it] = v;
             ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
@@ -455,22 +460,24 @@ __global__ void normed_add_rmsnorm_vec4_kernel(const TX* __restrict__ x, const f
 }
 
 // x [n_rows_total, width] of type dtype; wx, w float32 [width]; res float32 [n_rows_total, width]; rows null (every
-// row, res updated) or int32 [n_out] (those rows, res untouched); y [n_out, width] of type dtype, or null with w.
-PB_API int pb_normed_add_rmsnorm(const void* x, const float* wx, float eps_x, float* res, const int32_t* rows, int n_out,
-                                 int n_rows_total, const float* w, void* y, int dtype, int width, float eps,
+// row, res updated) or int32 [n_out] (those rows, res untouched); y [n_out, width] of type dtype, or null with w; plus null
+// or float32 [n_rows_total, width], not with rows.
+PB_API int pb_normed_add_rmsnorm(const void* x, const float* wx, float eps_x, float* res, const float* plus, const int32_t* rows,
+                                 int n_out, int n_rows_total, const float* w, void* y, int dtype, int width, float eps,
                                  cudaStream_t stream) {
     PB_REQUIRE(n_out >= 0 && n_rows_total >= 0 && width > 0, "normed_add_rmsnorm: bad sizes");
     PB_REQUIRE(x && wx && res && (w == nullptr || y != nullptr), "normed_add_rmsnorm: null pointer");
     PB_REQUIRE(rows == nullptr ? n_out == n_rows_total : y != nullptr, "normed_add_rmsnorm: rows and outputs do not fit");
+    PB_REQUIRE(plus == nullptr || rows == nullptr, "normed_add_rmsnorm: a second addend joins whole streams only");
     if (n_out == 0) return 0;
     const int threads = norm_threads(width);
     const size_t esz = dtype == PB_BF16 ? 2 : 4;
-    if (width % 4 == 0 && width <= 4 * threads * 8 && pb_aligned(x, 4 * esz) && pb_aligned(wx, 16) && pb_aligned(res, 16) &&
+    if (width % 4 == 0 && width <= 4 * threads * 8 && pb_aligned(x, 4 * esz) && pb_aligned(wx, 16) && pb_aligned(res, 16) && pb_aligned(plus, 16) &&
         (w == nullptr || pb_aligned(w, 16)) && (y == nullptr || pb_aligned(y, 4 * esz))) {
         const int iters = (width / 4 + threads - 1) / threads;
 #define NA_VEC(IT)                                                                                                              \
     PB_DISPATCH_DTYPE(dtype, T, (pb_launch(normed_add_rmsnorm_vec4_kernel<T, T, IT>, dim3(n_out), dim3(threads), 0, stream, (const T*)x, wx, \
-                                           eps_x, res, rows, n_rows_total, w, (T*)y, width, eps)))
+                                           eps_x, res, plus, rows, n_rows_total, w, (T*)y, width, eps)))
         if (iters <= 2) NA_VEC(2);
         else if (iters <= 4) NA_VEC(4);
         else NA_VEC(8);
@@ -482,7 +489,7 @@ PB_API int pb_normed_add_rmsnorm(const void* x, const float* wx, float eps_x, fl
     const size_t smem = keep ? (size_t)width * sizeof(float) : 0;
     PB_DISPATCH_DTYPE(dtype, T,
         (pb_launch(normed_add_rmsnorm_kernel<T, T>, dim3(n_out), dim3(norm_threads(width)), smem, stream, (const T*)x, wx, eps_x,
-                   res, rows, n_rows_total, w, (T*)y, width, eps, keep)));
+                   res, plus, rows, n_rows_total, w, (T*)y, width, eps, keep)));
     PB_CHECK_LAUNCH("normed_add_rmsnorm");
     return 0;
 }

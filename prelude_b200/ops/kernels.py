@@ -83,10 +83,11 @@ def embed_sinusoid(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tens
 class Normed:
     """A sublayer's output that is normed before it joins the residual stream: the value is
     ``x / sqrt(mean(x^2) + eps) * weight`` (weight float32, as applied), not computed yet.  The fused residual
-    add takes it as it is and norms, adds and norms again in one pass, in float32."""
+    add takes it as it is and norms, adds and norms again in one pass, in float32.  x may itself be a sublayer's last
+    kernel still to run (``Pending``).  ``plus``: float32 rows that join the stream beside it, or None (``joined``)."""
 
-    def __init__(self, x: torch.Tensor, weight: torch.Tensor, eps: float):
-        self.x, self.weight, self.eps = x, weight, float(eps)
+    def __init__(self, x, weight: torch.Tensor, eps: float, plus: Optional[torch.Tensor] = None):
+        self.x, self.weight, self.eps, self.plus = x, weight, float(eps), plus
 
     @property
     def shape(self):
@@ -97,10 +98,23 @@ def normed_add_rmsnorm(x: "Normed", res: torch.Tensor, weight: Optional[torch.Te
                        rows: Optional[torch.Tensor] = None, sum_out: bool = False) -> Optional[torch.Tensor]:
     """res += norm(x) (in place, unless ``rows`` picks rows: then res is left alone); returns rmsnorm(res) * weight
     in ``out_dtype`` for every row, or for the chosen ones; with ``weight`` None only the sum is made, and with
-    ``sum_out`` it is also returned in ``out_dtype`` (for a sublayer that reads the stream itself)."""
-    xt = x.x.materialize(out_dtype) if isinstance(x.x, PartialSums) else x.x
-    _need(xt, "x", out_dtype)
+    ``sum_out`` it is also returned in ``out_dtype`` (for a sublayer that reads the stream itself).  What ``x`` carries as
+    ``plus`` joins the sum too."""
     _need(x.weight, "x.weight", torch.float32)
+    if x.plus is not None:
+        _need(x.plus, "plus", torch.float32)
+        if x.plus.shape != res.shape or rows is not None:
+            raise KernelLibraryError(f"normed_add_rmsnorm: {tuple(x.plus.shape)} beside residual {tuple(res.shape)}; whole streams only")
+    xt = x.x
+    if isinstance(xt, Pending):
+        if weight is not None:
+            y = xt.add_normed(x, res, weight, eps, out_dtype, rows)
+            if y is not None:
+                return y
+        xt = xt.resolve()
+    if isinstance(xt, PartialSums):
+        xt = xt.materialize(out_dtype)
+    _need(xt, "x", out_dtype)
     _need(res, "res", torch.float32)
     total, width = res.shape
     if tuple(xt.shape) != tuple(res.shape) or x.weight.numel() != width:
@@ -116,8 +130,8 @@ def normed_add_rmsnorm(x: "Normed", res: torch.Tensor, weight: Optional[torch.Te
         _need(weight, "weight", torch.float32)
     if weight is not None or sum_out:
         out = torch.empty((n_out, width), dtype=out_dtype, device=res.device)
-    check(_l.library().pb_normed_add_rmsnorm(xt.data_ptr(), x.weight.data_ptr(), x.eps, res.data_ptr(), _ptr(rows), n_out, total,
-                                             _ptr(weight), _ptr(out), dtype_code(out_dtype), width, float(eps), _stream()),
+    check(_l.library().pb_normed_add_rmsnorm(xt.data_ptr(), x.weight.data_ptr(), x.eps, res.data_ptr(), _ptr(x.plus), _ptr(rows), n_out,
+                                             total, _ptr(weight), _ptr(out), dtype_code(out_dtype), width, float(eps), _stream()),
           "normed_add_rmsnorm")
     return out
 
@@ -161,10 +175,24 @@ class Pending:
     def add_squash(self, res: torch.Tensor, squash: Squash, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None):
         return None
 
+    def add_normed(self, normed: "Normed", res: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                   rows: Optional[torch.Tensor] = None):
+        """The output normed, added and the sum normed (``normed_add_rmsnorm``) in the last kernel, or None."""
+        return None
+
 
 def settled(x):
     """x with its last kernel run, where that is still to come."""
     return x.resolve() if isinstance(x, Pending) else x
+
+
+def joined(delta, rows: torch.Tensor, res: torch.Tensor):
+    """``delta`` as it is to be added to the residual stream when the float32 ``rows`` join the stream too: carried along
+    to the fused add where ``delta`` has one that takes them, else added to the stream at once."""
+    if isinstance(delta, Normed) and delta.plus is None:
+        return Normed(delta.x, delta.weight, delta.eps, rows)
+    res += rows
+    return delta
 
 
 def add_squash(x, res: torch.Tensor, squash: Squash, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -395,6 +423,17 @@ def relu2_(x: torch.Tensor) -> torch.Tensor:
     return x
 
 
+def sigmoid_gate_(y: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """y[t, i] *= sigmoid(gate[t, i]) in place for [T, cols] views with dense rows (float32 arithmetic)."""
+    for t, name in ((y, "y"), (gate, "gate")):
+        _need(t, name, y.dtype, contiguous=False)
+        if t.dim() != 2 or t.stride(1) != 1 or t.shape != y.shape:
+            raise KernelLibraryError(f"sigmoid_gate: {name} {tuple(t.shape)} must be [tokens, {y.shape[-1]}] with dense rows")
+    check(_l.library().pb_sigmoid_gate_(y.data_ptr(), y.stride(0), gate.data_ptr(), gate.stride(0), dtype_code(y.dtype), y.shape[0], y.shape[1],
+                                        _stream()), "sigmoid_gate")
+    return y
+
+
 def gemm_ref(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
              out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """a [M, K] times w [N, K] transposed (+ bias) on the float32 units."""
@@ -575,22 +614,33 @@ def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def _route_vectors(correction: Optional[torch.Tensor], bias: Optional[torch.Tensor], E: int) -> None:
+    for v, name in ((correction, "correction"), (bias, "bias")):
+        if v is not None:
+            _need(v, name, torch.float32)
+            if v.numel() != E:
+                raise KernelLibraryError(f"moe_route: a {name} of {v.numel()} numbers for {E} experts")
+
+
+def _scoring(softmax: bool, softmax_chosen: bool) -> int:
+    return 2 if softmax_chosen else 1 if softmax else 0          # as the library numbers them
+
+
 def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, group_top: int, renormalize: bool,
-              correction: Optional[torch.Tensor] = None, softmax: bool = False, renormalize_eps: float = 0.0, scale: float = 1.0):
-    """float32 router logits [T, E] -> (experts int32 [T, top], weights float32 [T, top]).  Scores are the logits'
-    sigmoids, or with ``softmax`` their softmax; ``correction`` float32 [E] joins the scores for the choice (groups and
+              correction: Optional[torch.Tensor] = None, softmax: bool = False, renormalize_eps: float = 0.0, scale: float = 1.0,
+              bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False):
+    """float32 router logits [T, E] -> (experts int32 [T, top], weights float32 [T, top]).  ``bias`` float32 [E] is added to
+    the logits.  Scores are the logits' sigmoids, or with ``softmax`` their softmax, or with ``softmax_chosen`` the logits
+    themselves; ``correction`` float32 [E] joins the scores for the choice (groups and
     experts) only; the weights are the scores without it (with ``renormalize`` divided by their sum plus
-    ``renormalize_eps``) times ``scale``."""
+    ``renormalize_eps``; with ``softmax_chosen`` the softmax over the chosen experts' logits) times ``scale``."""
     _need(logits, "logits", torch.float32)
     T, E = logits.shape
-    if correction is not None:
-        _need(correction, "correction", torch.float32)
-        if correction.numel() != E:
-            raise KernelLibraryError(f"moe_route: a correction of {correction.numel()} numbers for {E} experts")
+    _route_vectors(correction, bias, E)
     ids = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    check(_l.library().pb_moe_route(logits.data_ptr(), _ptr(correction), T, E, top, groups, keep, group_top, 1 if softmax else 0,
-                                    1 if renormalize else 0, float(renormalize_eps), float(scale), ids.data_ptr(), weights.data_ptr(), _stream()),
+    check(_l.library().pb_moe_route(logits.data_ptr(), _ptr(correction), _ptr(bias), T, E, top, groups, keep, group_top,
+                                    _scoring(softmax, softmax_chosen), 1 if renormalize else 0, float(renormalize_eps), float(scale), ids.data_ptr(), weights.data_ptr(), _stream()),
           "moe_route")
     return ids, weights
 
@@ -603,15 +653,17 @@ def moe_route_few_takes(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def moe_route_few(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: int, group_top: int, renormalize: bool,
-                  correction: Optional[torch.Tensor] = None, softmax: bool = False, renormalize_eps: float = 0.0, scale: float = 1.0):
+                  correction: Optional[torch.Tensor] = None, softmax: bool = False, renormalize_eps: float = 0.0, scale: float = 1.0,
+                  bias: Optional[torch.Tensor] = None, softmax_chosen: bool = False):
     """``router_logits`` and ``moe_route`` in one kernel for a few tokens; the same numbers."""
     _cols(x, "x")
     T, Kdim = x.shape
     E = w.shape[0]
+    _route_vectors(correction, bias, E)
     ids = torch.empty((T, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=x.device)
-    check(_l.library().pb_moe_route_few(x.data_ptr(), x.stride(0), w.data_ptr(), dtype_code(x.dtype), Kdim, _ptr(correction), T, E, top, groups, keep,
-                                        group_top, 1 if softmax else 0, 1 if renormalize else 0, float(renormalize_eps), float(scale),
+    check(_l.library().pb_moe_route_few(x.data_ptr(), x.stride(0), w.data_ptr(), dtype_code(x.dtype), Kdim, _ptr(correction), _ptr(bias), T, E, top,
+                                        groups, keep, group_top, _scoring(softmax, softmax_chosen), 1 if renormalize else 0, float(renormalize_eps), float(scale),
                                         ids.data_ptr(), weights.data_ptr(), _stream()), "moe_route_few")
     return ids, weights
 
@@ -641,20 +693,22 @@ def moe_sort(ids: torch.Tensor, n_experts: int, tile_rows: Optional[int] = None)
     return plan
 
 
-ACT_NONE, ACT_RELU, ACT_RELU2 = 0, 3, 4          # activations of the products' epilogues, as the library numbers them
+# activations of the products' epilogues, as the library numbers them (gated products: ACT_NONE is the SiLU gate)
+ACT_NONE, ACT_CLAMPED, ACT_RELU, ACT_RELU2 = 0, 1, 3, 4
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated: bool, gather_div: int = 0,
-             out_dtype: Optional[torch.dtype] = None, few_rows: bool = False, act: int = ACT_NONE) -> torch.Tensor:
+             out_dtype: Optional[torch.dtype] = None, few_rows: bool = False, act: int = ACT_NONE, limit: float = 0.0,
+             alpha: float = 0.0) -> torch.Tensor:
     """The experts' products over the plan's places.  a [rows, K]; w [E, N (2 N when gated: gate rows, then up rows), K];
     row of place p is ``order[p] // gather_div`` (the token of a slot) or, with gather_div 0, p itself.  Returns
-    [places, N]: a W_e^T (``act`` ACT_RELU2: its squared ReLU), or silu(a Wg_e^T) * (a Wu_e^T).  ``few_rows``: the
-    experts have a row or a few each (a decode
+    [places, N]: a W_e^T (``act`` ACT_RELU2: its squared ReLU), or silu(a Wg_e^T) * (a Wu_e^T), or (``act`` ACT_CLAMPED) the
+    clamped unit of the two with ``limit`` and ``alpha``.  ``few_rows``: the experts have a row or a few each (a decode
     step): the kernel that only streams the weights, where it takes the operands (bfloat16, K in multiples of 8)."""
     _cols(a, "a")
     _need(w, "w", a.dtype)
     E, rows_w, Kdim = w.shape
-    if a.shape[1] != Kdim or (gated and (rows_w % 2 or act)):
+    if a.shape[1] != Kdim or (gated and (rows_w % 2 or act not in (ACT_NONE, ACT_CLAMPED))):
         raise KernelLibraryError(f"moe_gemm: a {tuple(a.shape)} against w {tuple(w.shape)}")
     N = rows_w // 2 if gated else rows_w
     out_dtype = out_dtype or a.dtype
@@ -665,12 +719,12 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated: bool, gathe
     if (few_rows and plan.tile_rows == 64 and a.dtype == torch.bfloat16 and Kdim % 8 == 0 and a.stride(0) % 8 == 0
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
         check(_l.library().pb_moe_gemv(a.data_ptr(), a.stride(0), plan.order.data_ptr() if gather_div else None, max(1, gather_div),
-                                       w.data_ptr(), w.stride(0), N, Kdim, 1 if gated else 0, act, plan.tile_expert.data_ptr(),
+                                       w.data_ptr(), w.stride(0), N, Kdim, 1 if gated else 0, act, float(limit), float(alpha), plan.tile_expert.data_ptr(),
                                        plan.tile_row0.data_ptr(), plan.offsets.data_ptr(), plan.max_tiles, None, 0, out.data_ptr(), out.stride(0),
                                        dtype_code(out_dtype), _stream()), "moe_gemv")
         return out
     check(_l.library().pb_moe_gemm(a.data_ptr(), a.stride(0), plan.order.data_ptr() if gather_div else None, max(1, gather_div),
-                                   w.data_ptr(), w.stride(0), N, Kdim, 1 if gated else 0, act, plan.tile_expert.data_ptr(),
+                                   w.data_ptr(), w.stride(0), N, Kdim, 1 if gated else 0, act, float(limit), float(alpha), plan.tile_expert.data_ptr(),
                                    plan.tile_row0.data_ptr(), plan.offsets.data_ptr(), plan.max_tiles, plan.tile_rows, out.data_ptr(), out.stride(0),
                                    dtype_code(a.dtype), dtype_code(out_dtype), _stream()), "moe_gemm")
     return out
@@ -686,7 +740,7 @@ def moe_gemv_takes(a: torch.Tensor, w: torch.Tensor, n_slots: int) -> bool:
 
 
 def moe_gemv(a: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, rows_are_slots: bool, out_dtype: torch.dtype, gated: bool = False,
-             act: int = ACT_NONE) -> torch.Tensor:
+             act: int = ACT_NONE, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """The experts' products for a few tokens without a plan: ids int32 [T, top]; a [T, K] (the tokens' rows) or, with
     ``rows_are_slots``, [T * top, K]; the result's rows are the slots token * top + choice."""
     _cols(a, "a")
@@ -699,7 +753,7 @@ def moe_gemv(a: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, rows_are_slots
     N = rows_w // 2 if gated else rows_w
     out = torch.empty((T * top, N), dtype=out_dtype, device=a.device)
     check(_l.library().pb_moe_gemv(a.data_ptr(), a.stride(0), None, 1 if rows_are_slots else top, w.data_ptr(), w.stride(0), N, Kdim,
-                                   1 if gated else 0, act, None, None, None, E, ids.data_ptr(), T * top, out.data_ptr(), out.stride(0),
+                                   1 if gated else 0, act, float(limit), float(alpha), None, None, None, E, ids.data_ptr(), T * top, out.data_ptr(), out.stride(0),
                                    dtype_code(out_dtype), _stream()), "moe_gemv")
     return out
 
@@ -715,7 +769,7 @@ def moe_gather_rows(x: torch.Tensor, plan: MoePlan, div: int) -> torch.Tensor:
 
 
 def moe_gemm_pair(a_sorted: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated: bool, status: torch.Tensor,
-                  max_pairs: int = 0, act: int = ACT_NONE) -> torch.Tensor:
+                  max_pairs: int = 0, act: int = ACT_NONE, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """The experts' products on the paired-block tcgen05 kernel: a_sorted [places, K] bfloat16 holds the rows in the
     order of their places (``moe_gather_rows``), the plan has row tiles of 256; w as for ``moe_gemm``.  bfloat16 out."""
     _need(a_sorted, "a_sorted", torch.bfloat16)
@@ -727,7 +781,7 @@ def moe_gemm_pair(a_sorted: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated:
     out = torch.empty((a_sorted.shape[0], N), dtype=torch.bfloat16, device=a_sorted.device)
     check(_l.library().pb_gemm_pair_grouped_bf16(
         a_sorted.data_ptr(), w.data_ptr(), out.data_ptr(), a_sorted.shape[0], rows_w, E, Kdim, a_sorted.stride(0), Kdim,
-        out.stride(0), 1 if gated else 0, act, plan.tile_expert.data_ptr(), plan.tile_row0.data_ptr(), plan.offsets.data_ptr(),
+        out.stride(0), 1 if gated else 0, act, float(limit), float(alpha), plan.tile_expert.data_ptr(), plan.tile_row0.data_ptr(), plan.offsets.data_ptr(),
         plan.max_tiles, max_pairs, status.data_ptr(), _stream()), "gemm_pair (grouped)")
     return out
 
@@ -754,7 +808,8 @@ class PendingExperts(Pending):
         self.y, self.place_of, self.weights, self.shared, self.dtype = y, place_of, weights, shared, dtype
         self.shape = (weights.shape[0], y.shape[1])
 
-    def _run(self, res, squash: Optional[Squash], rows) -> torch.Tensor:
+    def _operands(self, res):
+        """(y .. shared's stride) as the library's sums take them, checked."""
         T, width = self.shape
         _need(self.y, "y")
         _need(self.weights, "weights", torch.float32)
@@ -768,11 +823,16 @@ class PendingExperts(Pending):
             raise KernelLibraryError(f"moe_sum: shared {tuple(sh.shape)} beside {(T, width)}")
         if res is not None and tuple(res.shape) != (T, width):
             raise KernelLibraryError(f"moe_sum: residual {tuple(res.shape)} against {(T, width)}")
+        return (self.y.data_ptr(), dtype_code(self.y.dtype), _ptr(self.place_of), self.weights.data_ptr(), _ptr(sh), dtype_code(sh_dtype),
+                parts, stride)
+
+    def _run(self, res, squash: Optional[Squash], rows) -> torch.Tensor:
+        T, width = self.shape
+        operands = self._operands(res)
         n_out = T if rows is None else rows.numel()
         out = torch.empty((n_out, width), dtype=self.dtype, device=self.y.device)
         check(_l.library().pb_moe_sum(
-            self.y.data_ptr(), dtype_code(self.y.dtype), _ptr(self.place_of), self.weights.data_ptr(), _ptr(sh), dtype_code(sh_dtype), parts, stride,
-            _ptr(res), _ptr(rows), squash.slope if squash else 0.0, _ptr(squash.weight) if squash else None, _ptr(squash.shift) if squash else None,
+            *operands, _ptr(res), _ptr(rows), squash.slope if squash else 0.0, _ptr(squash.weight) if squash else None, _ptr(squash.shift) if squash else None,
             out.data_ptr(), dtype_code(self.dtype), n_out, T, self.weights.shape[1], width, _stream()), "moe_sum")
         return out
 
@@ -781,6 +841,25 @@ class PendingExperts(Pending):
 
     def add_squash(self, res, squash, out_dtype, rows=None):
         return self._run(res, squash, rows) if out_dtype == self.dtype else None
+
+    def add_normed(self, normed, res, weight, eps, out_dtype, rows=None):
+        T, width = self.shape
+        if out_dtype != self.dtype or not _l.library().pb_moe_sum_normed_supported(width, dtype_code(self.dtype)):
+            return None
+        operands = self._operands(res)
+        _need(res, "res", torch.float32)
+        for v, name in ((normed.weight, "weight"), (weight, "weight of the norm that follows")):
+            _need(v, name, torch.float32)
+            if v.numel() != width:
+                raise KernelLibraryError(f"moe_sum_normed: {name} has {v.numel()} elements, rows have {width}")
+        if rows is not None:
+            _need(rows, "rows", torch.int32)
+        n_out = T if rows is None else rows.numel()
+        out = torch.empty((n_out, width), dtype=self.dtype, device=self.y.device)
+        check(_l.library().pb_moe_sum_normed(
+            *operands, normed.weight.data_ptr(), normed.eps, res.data_ptr(), _ptr(normed.plus), _ptr(rows), weight.data_ptr(), float(eps),
+            out.data_ptr(), dtype_code(self.dtype), n_out, T, self.weights.shape[1], width, _stream()), "moe_sum_normed")
+        return out
 
 
 # -- mixers whose norm spans more than a head, rotation by rates, general paged attention ---------------------------

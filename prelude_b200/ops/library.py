@@ -47,8 +47,8 @@ _SIGNATURES = {
     "pb_attention_prefill_tc_plain_pages_supported": ([I, I, I, I], I),
     "pb_attention_prefill_tc_masked_bf16": ([P, P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, F, P, P, L, P, P], I),
     "pb_attention_prefill_tc_rows_supported": ([I, I], I),
-    "pb_attention_prefill_tc_rows_bf16": ([P, P, P, P, I, I, P, P, P, P, P, P, I, I, I, I, I, F, P, P, L, P, P], I),
-    "pb_rows_gather_bf16": ([P, P, P, P, I, P, P, P, P, I, I, I, I, P, P], I),
+    "pb_attention_prefill_tc_rows_bf16": ([P, P, P, P, I, I, P, P, P, P, P, P, I, I, I, I, I, F, I, P, P, L, I, P, P], I),
+    "pb_rows_gather_bf16": ([P, P, P, P, I, P, P, P, P, I, I, I, I, P, I, P, P], I),
     "pb_attention_decode_scratch_floats": ([I, I, I, I], L),
     "pb_attention_decode_blocks_per_sm": ([I], I),
     "pb_attention_decode_bf16": ([P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, I, P, P, P, P], I),
@@ -69,7 +69,7 @@ _SIGNATURES = {
     "pb_gemm_pair_gelu_glu_bf16": ([P, P, P, I, I, I, L, L, L, I, P, P], I),
     "pb_embed_sinusoid": ([P, P, P, I, P, P, I, I, I, P], I),
     "pb_clamped_glu": ([P, P, I, I, I, F, F, P], I),
-    "pb_normed_add_rmsnorm": ([P, P, F, P, P, I, I, P, P, I, I, F, P], I),
+    "pb_normed_add_rmsnorm": ([P, P, F, P, P, P, I, I, P, P, I, I, F, P], I),
     "pb_kv_write_pages": ([P, L, P, L, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, P, P], I),
     "pb_diff_attention_ref": ([P, L, P, L, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, F, I, F, F, F, I, I, I, P, P], I),
     "pb_diff_attention_tc_supported": ([I, I, I, I, L], I),
@@ -77,14 +77,16 @@ _SIGNATURES = {
     "pb_diff_attention_tc_max_splits": ([I, I], I),
     "pb_diff_attention_tc_bf16": ([P, L, P, L, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, I, F, F, F, I, I, I, I, I, P, P, P], I),
     "pb_router_logits": ([P, L, P, P, I, I, I, I, P], I),
-    "pb_moe_route": ([P, P, I, I, I, I, I, I, I, I, F, F, P, P, P], I),
+    "pb_moe_route": ([P, P, P, I, I, I, I, I, I, I, I, F, F, P, P, P], I),
     "pb_moe_route_few_supported": ([I, I, I], I),
-    "pb_moe_route_few": ([P, L, P, I, I, P, I, I, I, I, I, I, I, I, F, F, P, P, P], I),
+    "pb_moe_route_few": ([P, L, P, I, I, P, P, I, I, I, I, I, I, I, I, F, F, P, P, P], I),
     "pb_moe_sum": ([P, I, P, P, P, I, I, L, P, P, F, P, P, P, I, I, I, I, I, P], I),
+    "pb_moe_sum_normed_supported": ([I, I], I),
+    "pb_moe_sum_normed": ([P, I, P, P, P, I, I, L, P, F, P, P, P, P, F, P, I, I, I, I, I, P], I),
     "pb_moe_tile_rows": ([I, I], I),
     "pb_moe_sort": ([P, I, I, P, P, P, P, P, I, I, P], I),
-    "pb_moe_gemm": ([P, L, P, I, P, L, I, I, I, I, P, P, P, I, I, P, L, I, I, P], I),
-    "pb_moe_gemv": ([P, L, P, I, P, L, I, I, I, I, P, P, P, I, P, I, P, L, I, P], I),
+    "pb_moe_gemm": ([P, L, P, I, P, L, I, I, I, I, F, F, P, P, P, I, I, P, L, I, I, P], I),
+    "pb_moe_gemv": ([P, L, P, I, P, L, I, I, I, I, F, F, P, P, P, I, P, I, P, L, I, P], I),
     "pb_moe_combine": ([P, I, P, P, P, I, I, I, I, P], I),
     "pb_moe_gather_rows": ([P, L, P, I, P, I, I, I, P], I),
     "pb_gemm_ref_batched": ([P, P, P, I, I, I, I, I, L, L, L, I, L, L, L, P], I),
@@ -103,13 +105,14 @@ _SIGNATURES = {
     "pb_silu_cols": ([P, L, I, I, I, P], I),
     "pb_gelu_tanh_mul": ([P, P, I, I, I, P], I),
     "pb_scaled_sum": ([P, F, P, F, P, I, I, L, P], I),
-    "pb_gemm_pair_grouped_bf16": ([P, P, P, I, I, I, I, L, L, L, I, I, P, P, P, I, I, P, P], I),
+    "pb_gemm_pair_grouped_bf16": ([P, P, P, I, I, I, I, L, L, L, I, I, F, F, P, P, P, I, I, P, P], I),
     "pb_gemm_pair_act_bf16": ([P, P, P, I, I, I, L, L, L, I, I, I, P, P], I),
     "pb_gemm_stream_act_bf16": ([P, P, P, I, I, I, L, L, L, I, I, I, P, P], I),
     "pb_gemm_stream_add_tanh_bf16": ([P, P, P, F, P, P, P, I, I, I, L, L, P, P], I),
     "pb_add_tanh": ([P, I, L, P, P, I, I, F, P, P, P, I, I, P], I),
     "pb_relu_mul": ([P, P, I, I, I, P], I),
     "pb_relu2_": ([P, I, L, P], I),
+    "pb_sigmoid_gate_": ([P, L, P, L, I, I, I, P], I),
     "pb_channel_decay": ([P, L, P, P, F, P, I, I, I, I, P], I),
     "pb_gla_scan": ([P, P, P, L, I, P, F, P, P, P, P, I, I, I, I, P], I),
     "pb_gla_step_supported": ([I, I], I),

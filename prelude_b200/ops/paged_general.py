@@ -120,34 +120,41 @@ ROWS_MAX = int(os.environ.get("PRELUDE_LATENT_ROWS_MAX", str(1 << 16)))
 
 class RowsPlan:
     """Which blocks of 128 dense rows a step's long portions need: block b holds positions ``block_pos0[b]`` .. of request
-    ``block_seq[b]``; ``row_blocks`` [requests, stride] lists a request's blocks (0 where it has none)."""
+    ``block_seq[b]``; ``row_blocks`` [requests, stride] lists a request's blocks by position / 128 (0 where it has none, also
+    for blocks that the window has passed)."""
 
-    def __init__(self, block_seq, block_pos0, row_blocks, n_blocks: int, all_long: bool):
+    def __init__(self, block_seq, block_pos0, row_blocks, n_blocks: int, all_long: bool, window: Optional[int] = None):
         self.block_seq, self.block_pos0, self.row_blocks, self.n_blocks, self.all_long = block_seq, block_pos0, row_blocks, n_blocks, all_long
+        self.window = window
 
 
-def rows_plan(batch) -> Optional[RowsPlan]:
-    """The plan of a step's portions of ``ROWS_MIN_PORTION`` tokens and more (made once per step), or None where there is none
-    or their contexts together have more than ``ROWS_MAX`` tokens."""
-    if "rows_plan" in batch.extras:
-        return batch.extras["rows_plan"]
+def rows_plan(batch, window: Optional[int] = None) -> Optional[RowsPlan]:
+    """The plan of a step's portions of ``ROWS_MIN_PORTION`` tokens and more (made once per step and window), or None where
+    there is none or the tokens they see together are more than ``ROWS_MAX``."""
+    key = ("rows_plan", window) if window else "rows_plan"
+    if key in batch.extras:
+        return batch.extras[key]
     plan = None
     lens, ctx = np.asarray(batch.q_lens), np.asarray(batch.kv_len_host)
     long = np.nonzero(lens >= ROWS_MIN_PORTION)[0]
-    if long.size and int(ctx[long].sum()) <= ROWS_MAX:
-        blocks = -(-ctx[long] // ROW_BLOCK)
-        n, stride = int(blocks.sum()), int(blocks.max())
+    first = np.zeros(long.size, dtype=np.int64)              # the first block that a token of the portion sees
+    if window:
+        first = np.maximum(np.asarray(batch.q_start_host)[long] - window + 1, 0) // ROW_BLOCK
+    if long.size and int((ctx[long] - first * ROW_BLOCK).sum()) <= ROWS_MAX:
+        ends = -(-ctx[long] // ROW_BLOCK)
+        n, stride = int((ends - first).sum()), int(ends.max())
         host = np.zeros(2 * n + lens.shape[0] * stride, dtype=np.int32)
         table = host[2 * n:].reshape(lens.shape[0], stride)
         at = 0
-        for r, k in zip(long.tolist(), blocks.tolist()):
+        for r, b0, b1 in zip(long.tolist(), first.tolist(), ends.tolist()):
+            k = b1 - b0
             host[at:at + k] = r
-            host[n + at:n + at + k] = np.arange(k, dtype=np.int32) * ROW_BLOCK
-            table[r, :k] = np.arange(at, at + k, dtype=np.int32)
+            host[n + at:n + at + k] = np.arange(b0, b1, dtype=np.int32) * ROW_BLOCK
+            table[r, b0:b1] = np.arange(at, at + k, dtype=np.int32)
             at += k
         dev = torch.from_numpy(host).to(batch.token_ids.device, non_blocking=True)
-        plan = RowsPlan(dev[:n], dev[n:2 * n], dev[2 * n:].view(lens.shape[0], stride), n, bool((lens >= ROWS_MIN_PORTION).all()))
-    batch.extras["rows_plan"] = plan
+        plan = RowsPlan(dev[:n], dev[n:2 * n], dev[2 * n:].view(lens.shape[0], stride), n, bool((lens >= ROWS_MIN_PORTION).all()), window)
+    batch.extras[key] = plan
     return plan
 
 
@@ -157,7 +164,7 @@ def rows_supported(kd: int, vd: int, row: int) -> bool:
 
 def gather_rows(pages: torch.Tensor, batch, group: int, plan: RowsPlan) -> torch.Tensor:
     """The cached rows of the plan's blocks out of ``pages`` [num_pages, 1, page_size, width]: [blocks * 128, width], zeros behind
-    a request's last token."""
+    a request's last token and where the plan's window has passed."""
     num_pages, one, page_size, width = pages.shape
     if one != 1 or pages.dtype != torch.bfloat16:
         raise _l.KernelLibraryError("gather_rows: one head of bfloat16 rows")
@@ -166,22 +173,26 @@ def gather_rows(pages: torch.Tensor, batch, group: int, plan: RowsPlan) -> torch
     check(_l.library().pb_rows_gather_bf16(
         pages.data_ptr(), out.data_ptr(), plan.block_seq.data_ptr(), plan.block_pos0.data_ptr(), plan.n_blocks, batch.kv_len.data_ptr(),
         batch.cu_q.data_ptr(), batch.table_row_of_token.data_ptr(), table.data_ptr(), table.shape[1], page_size, num_pages, width,
-        batch.status.data_ptr(), _l.current_stream_ptr(out.device)), "rows_gather")
+        batch.q_start.data_ptr(), int(plan.window or 0), batch.status.data_ptr(), _l.current_stream_ptr(out.device)), "rows_gather")
     return out
 
 
 def attention_rows(q: torch.Tensor, kv: torch.Tensor, value_dim: int, batch, plan: RowsPlan, scale: float, sink: Optional[torch.Tensor],
                    gate: Optional[torch.Tensor], out: torch.Tensor) -> torch.Tensor:
-    """Causal attention of the plan's long portions over dense rows: q [T, H, kd], kv [blocks * 128, H * (kd + value_dim)] (a
-    head's key before its value), out [T, H, value_dim] (the other portions' rows are left alone); the tcgen05 prompt kernel."""
+    """Causal attention of the plan's long portions over dense rows (inside the plan's window): q [T, H, kd], kv [blocks * 128,
+    H * (kd + value_dim)] (a head's key before its value), out [T, H, value_dim] (the other portions' rows are left alone); the
+    tcgen05 prompt kernel.  ``gate``: columns [T, H], a number a head, or [T, H * value_dim], one an element, or None."""
     T, H, kd = q.shape
     lib = _l.library()
     if kv.shape != (plan.n_blocks * ROW_BLOCK, H * (kd + value_dim)) or tuple(out.shape) != (T, H, value_dim) or not kv.is_contiguous():
         raise _l.KernelLibraryError(f"attention_rows: q {tuple(q.shape)}, rows {tuple(kv.shape)}, out {tuple(out.shape)}")
+    if gate is not None and tuple(gate.shape) not in ((T, H), (T, H * value_dim)):
+        raise _l.KernelLibraryError(f"attention_rows: a gate {tuple(gate.shape)} for {T} tokens, {H} heads of {value_dim}")
     tile_seq, tile_tok0, n_tiles = _prefill_plan(batch, 256, ROWS_MIN_PORTION, None)
     check(lib.pb_attention_prefill_tc_rows_bf16(
         q.data_ptr(), kv.data_ptr(), out.data_ptr(), plan.row_blocks.data_ptr(), plan.row_blocks.shape[1], plan.n_blocks,
         batch.positions.data_ptr(), batch.token_seq.data_ptr(), batch.cu_q.data_ptr(), batch.q_start.data_ptr(), tile_seq.data_ptr(),
-        tile_tok0.data_ptr(), n_tiles, T, H, kd, value_dim, float(scale), K._ptr(sink), K._ptr(gate), 0 if gate is None else gate.stride(0),
+        tile_tok0.data_ptr(), n_tiles, T, H, kd, value_dim, float(scale), int(plan.window or 0), K._ptr(sink), K._ptr(gate),
+        0 if gate is None else gate.stride(0), 0 if gate is None or gate.shape[1] == H else 1,
         batch.status.data_ptr(), _l.current_stream_ptr(q.device)), "attention_prefill_tc (rows)")
     return out

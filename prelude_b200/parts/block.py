@@ -83,7 +83,8 @@ class SandwichResidualBlock:
 
     The norm after a sublayer and the add and norm that follow are one kernel: what this block returns is its
     feed-forward's output with ``norm2b`` still to be applied (``kernels.Normed``), which the next block's first
-    norm, or the model's final norm, applies while it adds.  A block without a feed-forward returns its mixer's
+    norm, or the model's final norm, applies while it adds.  A feed-forward whose last kernel can do all of that as
+    well (the sum over routed experts) hands it on unrun (``kernels.Pending``).  A block without a feed-forward returns its mixer's
     output the same way.
     """
 
@@ -100,6 +101,8 @@ class SandwichResidualBlock:
             self.ff_norm = make_part("norm", spec.ff_norm, f"{p}.{spec.ff_norm_name}")
             self.feed_forward = make_part("feed_forward", spec.feed_forward, f"{p}.{spec.ff_name}")
             self.ff_post_norm = make_part("norm", spec.ff_post_norm, f"{p}.{spec.ff_post_norm_name}")
+            if hasattr(self.feed_forward, "defer_output"):
+                self.feed_forward.defer_output = True
 
     def parts(self):
         return tuple(x for x in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.ff_norm, self.feed_forward,

@@ -11,12 +11,14 @@ That is the way of decode steps and short portions.  A long prompt portion has m
 there it pays to make keys and values per head once: the context's rows are gathered from their pages, ONE product makes
 every head's [plain key | rotated key part | value] of them (the rotated part through rows of the identity, which copies
 it exactly), and the tcgen05 prompt kernel attends with keys of ``head_dim + rot_dim`` and values of ``value_dim``
-elements instead of rows of ``kv_rank + rot_dim`` and ``kv_rank`` (PRELUDE_LATENT_EXPAND=0 turns it off).
+elements instead of rows of ``kv_rank + rot_dim`` and ``kv_rank`` (PRELUDE_LATENT_EXPAND=0 turns it off).  With a window only
+the rows that the portion sees are gathered.
 
 Steps: down projections of queries and of latent + key part; norm of the query latent; up projection of the
 queries (or, for queries that come from the input directly, one merged projection [queries | latent + key part | gate]);
 one kernel norms the latent, rotates the key part and the queries' rotated part and writes the page;
-queries into latent space; attention with the sink and the gate per head; values out of latent space; output projection.
+queries into latent space; attention with the sink and the gate per head; values out of latent space (a gate per element
+multiplies them there); output projection.
 A layer that reads another layer's cache (``share_cache``) has no down projection of its own and writes nothing.
 """
 from __future__ import annotations
@@ -47,7 +49,10 @@ class LatentAttention:
             raise ValueError("this mixer takes a position encoding given by rates (kind 'rotary_rates')")
         if self.position.rotary_dim > spec.rot_dim:
             raise ValueError(f"a rotation of {self.position.rotary_dim} elements does not fit the rotated part of {spec.rot_dim}")
+        if spec.head_gate and spec.element_gate:
+            raise ValueError("the output's gate is one per head or one per element, not both")
         self.q_dim = spec.head_dim + spec.rot_dim
+        self.g_cols = spec.num_heads * spec.value_dim if spec.element_gate else spec.num_heads if spec.head_gate else 0
         self.row = spec.kv_rank + spec.rot_dim                  # what a token keeps in the cache
         self.w_dq = self.w_uq = self.w_dkv = self.w_uk_t = self.w_uv = self.w_o = None
         self.dq_norm = self.dkv_norm = self.sink = None
@@ -80,8 +85,8 @@ class LatentAttention:
             f"{p}.{s.uv_name}": TensorReq((s.num_heads * s.value_dim, s.kv_rank)),
             f"{p}.{s.o_name}": TensorReq((s.hidden_size, s.num_heads * s.value_dim)),
         })
-        if s.head_gate:
-            req[f"{p}.{s.gate_name}"] = TensorReq((s.num_heads, s.hidden_size))
+        if self.g_cols:
+            req[f"{p}.{s.gate_name}"] = TensorReq((self.g_cols, s.hidden_size))
         if s.sink:
             req[f"{p}.{s.sink_name}"] = TensorReq((s.num_heads,), "bias")
         return req
@@ -97,7 +102,7 @@ class LatentAttention:
 
         self.w_o = mat(s.o_name)
         if s.q_rank is None:
-            mats = [mat(s.q_name)] + ([mat(s.dkv_name)] if self.owns_latent else []) + ([mat(s.gate_name)] if s.head_gate else [])
+            mats = [mat(s.q_name)] + ([mat(s.dkv_name)] if self.owns_latent else []) + ([mat(s.gate_name)] if self.g_cols else [])
             pad = (-sum(m.shape[0] for m in mats)) % 8         # rows of the merged projection stay 16-byte aligned
             if pad:
                 mats.append(torch.zeros((pad, s.hidden_size), dtype=ctx.dtype, device=ctx.device))
@@ -107,7 +112,7 @@ class LatentAttention:
             self.dq_norm = vec(s.dq_name + s.norm_suffix)
             if self.owns_latent:
                 self.w_dkv = mat(s.dkv_name)
-            if s.head_gate:
+            if self.g_cols:
                 self.w_gate = mat(s.gate_name)
         if self.owns_latent:
             self.dkv_norm = vec(s.dkv_name + s.norm_suffix)
@@ -117,7 +122,7 @@ class LatentAttention:
         if s.sink:
             self.sink = vec(s.sink_name)
         self.position.load(get, ctx)
-        if EXPAND and ctx.dtype == torch.bfloat16 and s.window is None and rows_supported(self.q_dim, s.value_dim, self.row):
+        if EXPAND and ctx.dtype == torch.bfloat16 and rows_supported(self.q_dim, s.value_dim, self.row):
             w = torch.zeros((s.num_heads, self.q_dim + s.value_dim, self.row), dtype=ctx.dtype, device=ctx.device)
             w[:, :s.head_dim, :s.kv_rank] = self.w_uk_t.transpose(1, 2)
             w[:, s.head_dim:self.q_dim, s.kv_rank:] = torch.eye(s.rot_dim, dtype=ctx.dtype, device=ctx.device)
@@ -127,7 +132,7 @@ class LatentAttention:
     def activation_bytes_per_token(self, elem: int) -> int:
         s = self.spec
         rows = 0 if self.w_rows is None else s.num_heads * (2 * self.q_dim + s.value_dim) + self.row
-        return ((s.q_rank or 0) * 2 + rows + s.num_heads * (2 * self.q_dim + 2 * self.row + s.value_dim) + self.row) * elem + s.hidden_size * elem
+        return ((s.q_rank or 0) * 2 + rows + s.num_heads * (2 * self.q_dim + 2 * self.row + s.value_dim) + self.row + self.g_cols) * elem + s.hidden_size * elem
 
     def cache_need(self) -> KvPagesNeed:
         return KvPagesNeed(1, self.row, self.spec.window, v_heads=0, v_head_dim=0)
@@ -148,7 +153,7 @@ class LatentAttention:
         recorder = batch.extras.get("recorder")
         if self.w_rows is None or batch.decode_only or batch.max_q_len < ROWS_MIN_PORTION or recorder is not None:
             return None
-        return rows_plan(batch)
+        return rows_plan(batch, self.spec.window)
 
     def _in_latent_space(self, q, ckv, gate, batch, cache, below, o) -> None:
         """Attention against the cached rows as they are; portions of ``below`` tokens and more are left out."""
@@ -160,9 +165,11 @@ class LatentAttention:
         # queries into latent space, head by head: q_lat[:, h, :kv_rank] = q_plain[:, h] W_uk,h
         batched_linear(q_plain.transpose(0, 1), self.w_uk_t, q_lat.transpose(0, 1)[:, :, :s.kv_rank])
         o_lat = attention_general(q_lat, cache.k_pages, None, s.kv_rank, batch, cache.group, s.softmax_scale, s.window, self.sink,
-                                  out=batch.workspace("latent_o", (T, H, s.kv_rank), q.dtype), gate=gate, below=below)
+                                  out=batch.workspace("latent_o", (T, H, s.kv_rank), q.dtype), gate=gate if s.head_gate else None, below=below)
         # values out of latent space: o[:, h] = o_lat[:, h] W_uv,h^T
         batched_linear(o_lat.transpose(0, 1), self.w_uv, o.transpose(0, 1))
+        if s.element_gate:
+            K.sigmoid_gate_(o.view(T, H * s.value_dim), gate)
 
     def forward(self, x: torch.Tensor, batch, cache, write_cache: bool = True) -> torch.Tensor:
         s = self.spec
@@ -173,13 +180,13 @@ class LatentAttention:
             q = proj[:, :H * self.q_dim]                                  # [T, H * (head_dim + rot_dim)]
             c0 = H * self.q_dim + (self.row if self.owns_latent else 0)
             ckv = proj[:, H * self.q_dim:c0] if write_cache else None     # [T, kv_rank + rot_dim]
-            if s.head_gate:
-                gate = proj[:, c0:c0 + H]
+            if self.g_cols:
+                gate = proj[:, c0:c0 + self.g_cols]
         else:
             cq = K.rmsnorm(linear(x, self.w_dq), self.dq_norm, s.norm_eps)
             q = linear(cq, self.w_uq)
             ckv = linear(x, self.w_dkv) if write_cache else None
-            if s.head_gate:
+            if self.g_cols:
                 gate = linear(x, self.w_gate)
         o = batch.workspace("latent_values", (T, H, s.value_dim), x.dtype)
         plan = self._rows_plan(batch)

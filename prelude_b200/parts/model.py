@@ -126,8 +126,12 @@ class DecoderModel:
         ``batch.extras["recorder"]``; that is what lets a step be captured piece by piece."""
         with step_status(batch.status):
             res = self.embedding.forward(batch)
+            # ``res`` is updated in place: an order that adds the embedding's output again keeps a copy of it
+            start = res.clone() if any(c.adds_embedding for c in self.order) else None
             delta = None
             for call in self.order:
+                if call.adds_embedding:
+                    delta = K.joined(delta, start, res)
                 delta = self.blocks[call.block].forward(delta, res, batch, caches[call.cache], call.writes_cache)
         return delta, res
 

@@ -1,8 +1,9 @@
-"""Routed experts: a mixture of feed-forwards (SiLU-gated, or plain with squared ReLU), a few per token.
+"""Routed experts: a mixture of feed-forwards (SiLU-gated, gated by the clamped unit, or plain with squared ReLU), a few per token.
 
 The router's logits are a 32-bit product of the feed-forward's input with the
 router matrix (float32 sums of exact products on the float32 units, whatever
-the run's type: ``kernels.router_logits``).  Scores are their sigmoids or their softmax; experts form equal groups of
+the run's type: ``kernels.router_logits``), plus a bias where the design has one.  Scores are their sigmoids or their softmax,
+or the logits themselves with the softmax over the chosen ones as weights; experts form equal groups of
 neighbours, a group scores the sum of its largest scores, and only experts of
 the best groups can be chosen; the chosen scores weigh the experts' outputs
 (``RoutedExpertsSpec`` has the constants).  A learned correction per expert may
@@ -15,9 +16,10 @@ products over them (gate/up with the activation in the epilogue, then down)
 and a weighted sum per token: five launches after the router's product, none
 of whose shapes depends on what the router chose, so the part can be recorded.
 A decode step's few tokens take a shorter way: router product and choice in one
-kernel, no grouping (the products look an expert's rows up in the choices), and
-the weighted sum together with the residual add and the norm behind it where that
-norm can run there (``defer_output``).  Plain experts have up rows only in the
+kernel, no grouping (the products look an expert's rows up in the choices).
+The weighted sum runs together with what stands behind it where the block hands it
+on (``defer_output``): the residual add and a squashing, or the norm of the
+output, the add and the norm that follows.  Plain experts have up rows only in the
 first tensor.
 """
 from __future__ import annotations
@@ -41,6 +43,9 @@ ROUTE_FEW_TOKENS = int(os.environ.get("PRELUDE_MOE_ROUTE_FEW_TOKENS", "32"))
 # average rows per expert from which a step's products run on the paired-block tcgen05 kernel
 MOE_PAIR_MIN_ROWS = int(os.environ.get("PRELUDE_MOE_PAIR_MIN_ROWS", "192"))
 
+# an activation's name: (two matrices on the way up or one, its number in the products' epilogues)
+_ACTS = {"silu_gated": (True, K.ACT_NONE), "clamped_glu": (True, K.ACT_CLAMPED), "relu2": (False, K.ACT_RELU2)}
+
 
 @register_part("feed_forward", "routed_experts")
 class RoutedExperts:
@@ -48,16 +53,21 @@ class RoutedExperts:
 
     def __init__(self, spec: RoutedExpertsSpec, prefix: str):
         s = spec
-        if s.activation not in ("silu_gated", "relu2") or s.scoring not in ("sigmoid", "softmax"):
+        if s.activation not in _ACTS or s.scoring not in ("sigmoid", "softmax", "softmax_chosen"):
             raise ValueError(f"routed experts with activation {s.activation!r} and scores by {s.scoring!r} are not known")
-        self.gated = s.activation == "silu_gated"
-        self.act = K.ACT_NONE if self.gated else K.ACT_RELU2
+        if s.scoring == "softmax_chosen" and s.renormalize:
+            raise ValueError("weights that are a softmax over the chosen experts add up to one: nothing to renormalize")
+        self.gated, act = _ACTS[s.activation]
+        self.clamped = act == K.ACT_CLAMPED
+        if self.clamped and (s.limit <= 0 or (s.shared_size is not None and s.shared_limit <= 0)):
+            raise ValueError(f"the clamped unit needs a positive limit, got {s.limit} and {s.shared_limit} for the shared expert")
+        self.act = dict(act=act, limit=s.limit, alpha=s.alpha) if self.clamped else dict(act=act)
         if s.n_experts % s.n_groups or not 0 < s.keep_groups <= s.n_groups:
             raise ValueError(f"{s.n_experts} experts do not form {s.n_groups} equal groups of which {s.keep_groups} are kept")
         if not 0 < s.top_k <= s.keep_groups * (s.n_experts // s.n_groups):
             raise ValueError(f"top_k={s.top_k} experts cannot come from {s.keep_groups} groups of {s.n_experts // s.n_groups}")
         self.spec, self.prefix = spec, prefix
-        self.w_router = self.w_gate_up = self.w_down = self.correction = None
+        self.w_router = self.w_gate_up = self.w_down = self.correction = self.router_bias = None
         self.w_shared_up = self.w_shared_down = None
 
     def _expert(self, e: int, name: str) -> str:
@@ -68,6 +78,8 @@ class RoutedExperts:
         req = {f"{self.prefix}.{s.router_name}": TensorReq((s.n_experts, s.hidden_size))}
         if s.correction_name is not None:
             req[f"{self.prefix}.{s.correction_name}"] = TensorReq((s.n_experts,), "bias")
+        if s.router_bias_name is not None:
+            req[f"{self.prefix}.{s.router_bias_name}"] = TensorReq((s.n_experts,), "bias")
         every = [(f"{self.prefix}.{s.expert_prefix}{e}", s.expert_size) for e in range(s.n_experts)]
         if s.shared_size is not None:
             every.append((f"{self.prefix}.{s.shared_prefix}", s.shared_size))
@@ -85,8 +97,14 @@ class RoutedExperts:
             return get(name).to(device=ctx.device, dtype=ctx.dtype)
 
         self.w_router = mat(f"{self.prefix}.{s.router_name}").contiguous()
+
+        def vec(name):
+            return get(f"{self.prefix}.{name}").to(device=ctx.device, dtype=torch.float32).contiguous()
+
         if s.correction_name is not None:
-            self.correction = get(f"{self.prefix}.{s.correction_name}").to(device=ctx.device, dtype=torch.float32).contiguous()
+            self.correction = vec(s.correction_name)
+        if s.router_bias_name is not None:
+            self.router_bias = vec(s.router_bias_name)
 
         def up(name):
             rows = [mat(f"{name}.{s.gate_name}"), mat(f"{name}.{s.up_name}")] if self.gated else [mat(f"{name}.{s.up_name}")]
@@ -115,7 +133,7 @@ class RoutedExperts:
     def _router_args(self):
         s = self.spec
         return (s.top_k, s.n_groups, s.keep_groups, s.group_score_top, s.renormalize, self.correction, s.scoring == "softmax",
-                s.renormalize_eps, s.weight_scale)
+                s.renormalize_eps, s.weight_scale, self.router_bias, s.scoring == "softmax_chosen")
 
     def route(self, x: torch.Tensor):
         """(experts int32 [T, top_k], weights float32 [T, top_k]) for the rows of x."""
@@ -127,7 +145,12 @@ class RoutedExperts:
         """What every token adds beside its experts, or None."""
         if self.w_shared_up is None:
             return None
-        if self.gated:
+        s = self.spec
+        if self.clamped:
+            h = L.gated_linear_clamped(x, self.w_shared_up, s.shared_limit, s.alpha)
+            if h is None:
+                h = K.clamped_glu(L.linear(x, self.w_shared_up), s.shared_limit, s.alpha)
+        elif self.gated:
             h = L.gated_linear_silu(x, self.w_shared_up)
             if h is None:
                 h = K.silu_mul(L.linear(x, self.w_shared_up))
@@ -147,16 +170,16 @@ class RoutedExperts:
             # a long prompt step: rows sorted by expert, both products on the paired-block tcgen05 kernel (tiles of 256 rows)
             plan = K.moe_sort(ids, s.n_experts, 256)
             status = L.tc_status(x.device)
-            h = K.moe_gemm_pair(K.moe_gather_rows(x, plan, s.top_k), self.w_gate_up, plan, self.gated, status, act=self.act)
+            h = K.moe_gemm_pair(K.moe_gather_rows(x, plan, s.top_k), self.w_gate_up, plan, self.gated, status, **self.act)
             return self._sum(K.moe_gemm_pair(h, self.w_down, plan, False, status), plan.place_of, weights, shared, x.dtype)
         # tiles of 128 rows where the experts have many rows each and the tensor-core kernel takes the shapes, else of 64
         small = x.dtype != torch.bfloat16 or s.hidden_size % 8 or s.expert_size % 8
         few = not small and x.shape[0] * s.top_k <= MOE_FEW_ROWS * s.n_experts       # a decode step: stream the weights
         if few and K.moe_gemv_takes(x, self.w_gate_up, ids.numel()):
-            h = K.moe_gemv(x, self.w_gate_up, ids, False, x.dtype, gated=self.gated, act=self.act)
+            h = K.moe_gemv(x, self.w_gate_up, ids, False, x.dtype, gated=self.gated, **self.act)
             y = K.moe_gemv(h, self.w_down, ids, True, torch.float32)
             return self._sum(y, None, weights, shared, x.dtype)
         plan = K.moe_sort(ids, s.n_experts, 64 if (small or few) else None)
-        h = K.moe_gemm(x, self.w_gate_up, plan, gated=self.gated, gather_div=s.top_k, few_rows=few, act=self.act)
+        h = K.moe_gemm(x, self.w_gate_up, plan, gated=self.gated, gather_div=s.top_k, few_rows=few, **self.act)
         y = K.moe_gemm(h, self.w_down, plan, gated=False, out_dtype=torch.float32, few_rows=few)
         return self._sum(y, plan.place_of, weights, shared, x.dtype)

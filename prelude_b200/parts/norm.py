@@ -5,7 +5,7 @@ y = x / sqrt(mean(x^2) + eps) * w in float32
 crates/prelude-core/src/models/commons/linear.rs:435-501).  The scale is kept
 in float32 whatever the run's type: a bfloat16 scale converts exactly, and one
 stored in 32-bit keeps its bits.  A scale stored around zero (``NormSpec.offset`` 1)
-is kept as ``offset + w``, added once in float32 when the tensor is loaded.
+is kept as ``offset + w``, added once in float32 when the tensor is loaded, times ``NormSpec.gain``.
 
 What a norm adds to the residual stream may itself be waiting for a norm
 (``kernels.Normed``: the output of a sublayer that is normed before the add);
@@ -44,7 +44,9 @@ class RmsNorm:
 
     def load(self, get, ctx: RunContext) -> None:
         w = get(self.name).to(device=ctx.device, dtype=torch.float32)
-        self.weight = (w + float(self.spec.offset) if self.spec.offset else w).contiguous()
+        if self.spec.offset:
+            w = w + float(self.spec.offset)
+        self.weight = (w * float(self.spec.gain) if self.spec.gain != 1.0 else w).contiguous()
         self.dtype = ctx.dtype
 
     def pending(self, x) -> K.Normed:
