@@ -27,7 +27,8 @@ running decodes, 256 tokens each), as generated tokens a second by the wall cloc
 ``--workload pabelix`` and ``--workload kolisun`` put that design beside Qwen3 dense at equal
 layer sizes (random weights): prefill and decode steps, and the design's kernels beside their
 like, each a line of its own; ``--workload nedesun`` and ``--workload pepolorn`` do so beside Kolisun and
-Qwen3 dense, ``--workload nulilix`` beside Pepolorn, Kolisun and Qwen3 dense.
+Qwen3 dense, ``--workload nulilix`` beside Pepolorn, Kolisun and Qwen3 dense, ``--workload tudulix`` beside
+Nulilix, Kolisun and Qwen3 dense.
 None of them changes the default run or its line.
 """
 import argparse
@@ -1353,6 +1354,237 @@ def nulilix_compare(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------------------
+# --workload tudulix: the Tudulix design beside Nulilix (routed experts beside a shared one, attention through a latent),
+# Kolisun (window attention, attention through a latent) and Qwen3 dense at equal layer sizes
+# ---------------------------------------------------------------------------------------------------------------
+TUDULIX_SIZES = {
+    # width; window attention: heads, key/value heads, head size, rotated elements; latent attention: heads, plain and rotated
+    # query/key sizes, value size, latent size; both windows; routed experts: how many, how many per token, their width, the
+    # shared expert's width
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, rot_dims=64, lat_heads=16, lat_dim=128, rot=64, vdim=128, kv_rank=512, window=1024,
+               experts=32, top=4, expert_ff=2048, shared_ff=2048, ff=8192),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, rot_dims=64, lat_heads=32, lat_dim=128, rot=64, vdim=128, kv_rank=512, window=1024,
+               experts=64, top=6, expert_ff=2048, shared_ff=2048, ff=12288),
+}
+
+
+def tudulix_config(z, layers, vocab):
+    """Layers that resemble a real model's, ``layers`` layer runs in all: window attention and latent attention in turn, every
+    layer with routed experts and a shared one; the two layers behind the first run twice with the same weights."""
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+           "mask": {"size": z["window"]}, "rot": {"dims": z["rot_dims"], "base": 500000.0}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["rot"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+           "scale": (z["lat_dim"] + z["rot"]) ** -0.5, "mask": {"size": z["window"]}, "rot": {"dims": z["rot"], "base": 10000.0}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0}, "shared": {"ff": z["shared_ff"], "limit": 10.0},
+           "router": {"experts": z["experts"], "top": z["top"]}}
+    n = max(3, layers - 2)
+    out = [{"type": "latent_attention" if i % 2 else "attention", "mixer": lat if i % 2 else att, "mlp": moe} for i in range(n)]
+    return {"architecture": "Tudulix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "logit_scale": 0.5, "layers": out, "loop": {"start": 1, "stop": 3, "times": 2}}
+
+
+def tudulix_kernels(pk, size):
+    """The new design's kernels beside their like of the closest models, one launch each: both attentions over a window beside
+    Kolisun's and Qwen3's over everything; the kernel between projection and pages beside Kolisun's; the gate per element; the
+    sum over the experts with the norms beside Nulilix's with the squashing and beside separate kernels; the residual add with
+    two norms with and without the embedding's output; the router by the chosen logits beside the softmax one; the experts with
+    the clamped unit beside the SiLU-gated ones."""
+    import torch
+    from prelude_b200.cache.manager import CacheManager
+    from prelude_b200.engine.batch import StepItem, build_step_batch
+    from prelude_b200.ops import kernels as K
+    from prelude_b200.ops import linear as L
+    from prelude_b200.ops.attention import paged_attention
+    from prelude_b200.ops.paged_general import attention_general, attention_rows, gather_rows, rows_plan
+    from prelude_b200.parts.registry import KvPagesNeed
+    z = TUDULIX_SIZES[size]
+    dev = torch.device("cuda:0")
+    flush = torch.empty(160 << 20, dtype=torch.uint8, device=dev)
+    bf = torch.bfloat16
+    out = {}
+    T, B, ctx, win = 2048, 8, 2048, z["window"]
+    W, H, G, D = z["width"], z["heads"], z["kv"], z["dim"]
+    LH, rank, row, kd, vd = z["lat_heads"], z["kv_rank"], z["kv_rank"] + z["rot"], z["lat_dim"] + z["rot"], z["vdim"]
+    E, top, F, SF = z["experts"], z["top"], z["expert_ff"], z["shared_ff"]
+    cache = CacheManager([KvPagesNeed(1, row, None, 0, 0), KvPagesNeed(G, D)], PAGE_SIZE, (B * (ctx + 16) + T) // PAGE_SIZE + 8, B + 1, dev, bf)
+    lat, gqa = cache.layer_cache(0), cache.layer_cache(1)
+    lat.k_pages.normal_()
+    gqa.k_pages.normal_()
+    gqa.v_pages.normal_()
+    g0, g1 = cache.group_of[0], cache.group_of[1]
+    rnd = lambda *shape: torch.randn(*shape, device=dev).to(bf)
+    ones = lambda n: torch.ones(n, device=dev)
+
+    def both(name, unit, ours, theirs, reps=10):
+        """A launch and its likes by the model's name: (function, work in FLOPs or bytes) of each."""
+        entry = {}
+        for label, (fn, work) in {"ours": ours, **theirs}.items():
+            ms = _event_ms(fn, flush=flush, reps=reps)
+            entry[f"{label}_us"] = round(ms * 1e3, 2)
+            entry[f"{label}_{unit}"] = round(work / ms / (1e9 if unit == "tflops" else 1e6), 1)
+        out[name] = entry
+
+    # -- one request of T prompt tokens
+    cache.add_request("p")
+    cache.grow("p", T)
+    batch = build_step_batch([StepItem("p", [0] * T, 0, [])], cache.block_tables(["p"]), [cache.slot_of("p")], dev, 10, 1 << 20)
+    every = T * (T + 1) // 2
+    seen = sum(min(i + 1, win) for i in range(T))
+    q = rnd(T, H, D)
+    both("window_attention_prefill", "tflops",
+         (lambda: paged_attention(q, gqa.k_pages, gqa.v_pages, batch, g1, D ** -0.5, win), 4.0 * H * D * seen),
+         {"qwen3": (lambda: paged_attention(q, gqa.k_pages, gqa.v_pages, batch, g1, D ** -0.5, None), 4.0 * H * D * every)})
+    plan_w, plan = rows_plan(batch, win), rows_plan(batch)
+    w_rows = (torch.randn(LH * (kd + vd), row, device=dev) * 0.03).to(bf)
+    qf, of, gates, head_gates = rnd(T, LH, kd), torch.empty(T, LH, vd, dtype=bf, device=dev), rnd(T, LH * vd), rnd(T, LH)
+    kv = L.linear(gather_rows(lat.k_pages, batch, g0, plan), w_rows)
+    sink = torch.zeros(LH, device=dev)
+    both("latent_attention_prefill", "tflops",
+         (lambda: attention_rows(qf, kv, vd, batch, plan_w, kd ** -0.5, None, gates, of), 2.0 * LH * (kd + vd) * seen),
+         {"nulilix": (lambda: attention_rows(qf, kv, vd, batch, plan, kd ** -0.5, None, head_gates, of), 2.0 * LH * (kd + vd) * every),
+          "kolisun": (lambda: attention_rows(qf, kv, vd, batch, plan, kd ** -0.5, sink, None, of), 2.0 * LH * (kd + vd) * every)})
+    both("latent_rows_prefill", "gbs", (lambda: gather_rows(lat.k_pages, batch, g0, plan_w), 2.0 * T * row * 2),
+         {"kolisun": (lambda: gather_rows(lat.k_pages, batch, g0, plan), 2.0 * T * row * 2)})
+    ql = rnd(T, LH, row)
+    both("latent_space_prefill", "tflops",
+         (lambda: attention_general(ql, lat.k_pages, None, rank, batch, g0, kd ** -0.5, win, None), 2.0 * LH * (row + rank) * seen),
+         {"kolisun": (lambda: attention_general(ql, lat.k_pages, None, rank, batch, g0, kd ** -0.5, None, sink), 2.0 * LH * (row + rank) * every)})
+    proj = rnd(T, (H + 2 * G) * D)
+    rates, rates_all, qo = torch.rand(z["rot_dims"] // 2, device=dev), torch.rand(D // 2, device=dev), torch.empty(T, H, D, dtype=bf, device=dev)
+
+    def prepare(p, o, b, r, dims, wq, wk):
+        return K.qkv_prepare(p[:, :H * D], p[:, H * D:(H + G) * D], p[:, (H + G) * D:], n_heads=H, q_dim=D, q_weight=wq, k_weight=wk,
+                             k_norm_cols=G * D, eps=1e-6, rates=r, rot_dims=dims, adjacent=True, positions=b.positions,
+                             table_row=b.table_row_of_token, block_table=b.block_tables[g1], q_out=o, k_pages=gqa.k_pages, v_pages=gqa.v_pages,
+                             swizzle_k=True, swizzle_v=True, status=b.status)
+
+    wq, wk = ones(H * D), ones(G * D)
+    moved = T * (H + 2 * G) * D * 2 * 2.0
+    both("projection_to_pages_prefill", "gbs", (lambda: prepare(proj, qo, batch, rates, z["rot_dims"], None, None), moved),
+         {"kolisun": (lambda: prepare(proj, qo, batch, rates_all, D, wq, wk), moved)})
+    of2 = of.view(T, LH * vd)
+    both("gate_per_element_prefill", "gbs", (lambda: K.sigmoid_gate_(of2, gates), 3.0 * T * LH * vd * 2), {})
+    # residual add between two norms
+    res, x, emb, nw = torch.randn(T, W, device=dev), rnd(T, W), torch.randn(T, W, device=dev), ones(W)
+    both("residual_add_prefill", "gbs",
+         (lambda: K.normed_add_rmsnorm(K.Normed(x, nw, 1e-6, emb), res, nw, 1e-6, bf), T * W * (4.0 + 4 + 4 + 2 + 2)),
+         {"without_embedding": (lambda: K.normed_add_rmsnorm(K.Normed(x, nw, 1e-6), res, nw, 1e-6, bf), T * W * (4.0 + 4 + 2 + 2)),
+          "qwen3": (lambda: K.add_rmsnorm(x, res, nw, 1e-6, bf), T * W * (4.0 + 4 + 2 + 2))})
+    # routed experts
+    logits, bias, w_r = torch.randn(T, E, device=dev), torch.randn(E, device=dev), (torch.randn(E, W, device=dev) * 0.02).to(bf)
+    chosen, softmax = (top, 1, 1, 2, False, None, False, 0.0, 1.0, bias, True), (top, 4, 2, 1, True, None, True, 1e-20, 1.5)
+    both("router_choice_prefill", "gbs", (lambda: K.moe_route(logits, *chosen), T * E * 4.0), {"nulilix": (lambda: K.moe_route(logits, *softmax), T * E * 4.0)})
+    ids, weights = K.moe_route(logits, *chosen)
+    w_gu, w_dn = (torch.randn(E, 2 * F, W, device=dev) * 0.02).to(bf), (torch.randn(E, W, F, device=dev) * 0.02).to(bf)
+    status = L.tc_status(dev)
+    unit = dict(act=K.ACT_CLAMPED, limit=7.0, alpha=1.702)
+    splan = K.moe_sort(ids, E, 256)
+    xs = K.moe_gather_rows(x, splan, top)
+    h = K.moe_gemm_pair(xs, w_gu, splan, True, status, **unit)
+    y = K.moe_gemm_pair(h, w_dn, splan, False, status)
+    fl = 2.0 * T * top * F * W
+    both("experts_up_prefill", "tflops", (lambda: K.moe_gemm_pair(xs, w_gu, splan, True, status, **unit), 2 * fl),
+         {"pabelix": (lambda: K.moe_gemm_pair(xs, w_gu, splan, True, status), 2 * fl)})
+    both("experts_down_prefill", "tflops", (lambda: K.moe_gemm_pair(h, w_dn, splan, False, status), fl), {})
+    w_sh = (torch.randn(2 * SF, W, device=dev) * 0.02).to(bf)
+    fl = 2.0 * T * 2 * SF * W
+    both("shared_up_prefill", "tflops", (lambda: L.gated_linear_clamped(x, w_sh, 10.0, 1.702), fl), {"silu": (lambda: L.gated_linear_silu(x, w_sh), fl)})
+    sh = rnd(T, W)
+    pend, sq = K.PendingExperts(y, splan.place_of, weights, sh, bf), K.Squash(0.5, nw, torch.zeros(W, device=dev))
+    moved = T * W * (top * 2 + 2 + 8 + 2.0)
+    both("experts_sum_prefill", "gbs", (lambda: K.normed_add_rmsnorm(K.Normed(pend, nw, 1e-6), res, nw, 1e-6, bf), moved),
+         {"nulilix": (lambda: K.add_squash(pend, res, sq, bf), moved),
+          "separate": (lambda: K.normed_add_rmsnorm(K.Normed(pend.resolve(), nw, 1e-6), res, nw, 1e-6, bf), moved + T * W * 4.0)})
+    cache.release("p")
+    # -- B single tokens at ctx keys
+    rids = [f"d{i}" for i in range(B)]
+    for r in rids:
+        cache.add_request(r)
+        cache.grow(r, ctx + 1)
+    batch = build_step_batch([StepItem(r, [0], ctx, []) for r in rids], cache.block_tables(rids), [cache.slot_of(r) for r in rids], dev, 10, 1 << 20)
+    q8, l8, r8, x8, e8 = q[:B].contiguous(), ql[:B].contiguous(), res[:B].contiguous(), x[:B].contiguous(), emb[:B].contiguous()
+    few = dict(reps=20)
+    both("window_attention_decode", "gbs", (lambda: paged_attention(q8, gqa.k_pages, gqa.v_pages, batch, g1, D ** -0.5, win), B * win * G * D * 4.0),
+         {"qwen3": (lambda: paged_attention(q8, gqa.k_pages, gqa.v_pages, batch, g1, D ** -0.5, None), B * (ctx + 1) * G * D * 4.0)}, **few)
+    both("latent_attention_decode", "gbs", (lambda: attention_general(l8, lat.k_pages, None, rank, batch, g0, kd ** -0.5, win, None), B * win * row * 2.0),
+         {"kolisun": (lambda: attention_general(l8, lat.k_pages, None, rank, batch, g0, kd ** -0.5, None, sink), B * (ctx + 1) * row * 2.0)}, **few)
+    both("projection_to_pages_decode", "gbs", (lambda: prepare(proj[:B], qo[:B], batch, rates, z["rot_dims"], None, None), B * (H + 2 * G) * D * 4.0),
+         {"kolisun": (lambda: prepare(proj[:B], qo[:B], batch, rates_all, D, wq, wk), B * (H + 2 * G) * D * 4.0)}, **few)
+    w_uv, o_lat, o8, gates8 = rnd(LH, vd, rank), rnd(B, LH, rank), torch.empty(B, LH, vd, dtype=bf, device=dev), gates[:B].contiguous()
+    values = lambda: L.batched_linear(o_lat.transpose(0, 1), w_uv, o8.transpose(0, 1))
+    both("latent_values_decode", "gbs", (lambda: (values(), K.sigmoid_gate_(o8.view(B, LH * vd), gates8)), LH * vd * rank * 2.0),
+         {"kolisun": (values, LH * vd * rank * 2.0)}, **few)
+    both("residual_add_decode", "gbs", (lambda: K.normed_add_rmsnorm(K.Normed(x8, nw, 1e-6, e8), r8, nw, 1e-6, bf), B * W * 16.0),
+         {"qwen3": (lambda: K.add_rmsnorm(x8, r8, nw, 1e-6, bf), B * W * 12.0)}, **few)
+    both("router_decode", "gbs", (lambda: K.moe_route_few(x8, w_r, *chosen), E * W * 2.0), {"nulilix": (lambda: K.moe_route_few(x8, w_r, *softmax), E * W * 2.0)}, **few)
+    ids, weights = K.moe_route_few(x8, w_r, *chosen)
+    hit = int(torch.unique(ids).numel())
+    both("experts_up_decode", "gbs", (lambda: K.moe_gemv(x8, w_gu, ids, False, bf, gated=True, **unit), hit * 2 * F * W * 2.0),
+         {"silu": (lambda: K.moe_gemv(x8, w_gu, ids, False, bf, gated=True), hit * 2 * F * W * 2.0)}, **few)
+    h8 = K.moe_gemv(x8, w_gu, ids, False, bf, gated=True, **unit)
+    both("experts_down_decode", "gbs", (lambda: K.moe_gemv(h8, w_dn, ids, True, torch.float32), hit * F * W * 2.0), {}, **few)
+    out["experts_hit_decode"] = hit
+    both("shared_up_decode", "gbs", (lambda: L.gated_linear_clamped(x8, w_sh, 10.0, 1.702), 2 * SF * W * 2.0), {"silu": (lambda: L.gated_linear_silu(x8, w_sh), 2 * SF * W * 2.0)}, **few)
+    y8 = K.moe_gemv(h8, w_dn, ids, True, torch.float32)
+    pend8 = K.PendingExperts(y8, None, weights, sh[:B].contiguous(), bf)
+    moved = B * W * (top * 4 + 2 + 8 + 2.0)
+    both("experts_sum_decode", "gbs", (lambda: K.normed_add_rmsnorm(K.Normed(pend8, nw, 1e-6), r8, nw, 1e-6, bf), moved),
+         {"nulilix": (lambda: K.add_squash(pend8, r8, sq, bf), moved),
+          "separate": (lambda: K.normed_add_rmsnorm(K.Normed(pend8.resolve(), nw, 1e-6), r8, nw, 1e-6, bf), moved)}, **few)
+    if int(status.item()) != 0:
+        raise RuntimeError("a product raised the status word")
+    out["peaks"] = {"bf16_tflops": pk["bf16_tflops"], "hbm_gbs": pk["hbm_gbs"], "source": pk["source"]}
+    return out
+
+
+def tudulix_compare(args):
+    """Prefill and decode throughput of Tudulix beside Nulilix, Kolisun and Qwen3 dense at equal layer sizes and numbers of
+    layer runs (random weights, bfloat16): one prompt of --prefill-tokens through the step function, and --batch requests
+    decoding behind --prefix-len tokens on the captured step, both timed on the device.  One JSON line of its own."""
+    import torch
+    pk = peaks()
+    clocks = ClockSampler()
+    clocks.start()
+    t_begin = time.time()
+    points = []
+    vocab = 32768
+    for size in args.sizes.split(","):
+        z, layers = TUDULIX_SIZES[size], args.layers or 6
+        arms = {
+            "tudulix": tudulix_config(z, layers, vocab),
+            "nulilix": nulilix_config(NULILIX_SIZES[size], layers, vocab),
+            "kolisun": kolisun_config(KOLISUN_SIZES[size], layers, vocab),
+            "qwen3": dict(QWEN3_4B, vocab_size=vocab, hidden_size=z["width"], intermediate_size=z["ff"], num_hidden_layers=layers,
+                          num_attention_heads=z["heads"], num_key_value_heads=z["kv"], head_dim=z["dim"], tie_word_embeddings=True),
+        }
+        point = {"size": size, "layers": layers, "width": z["width"]}
+        for name, cfg in arms.items():
+            if args.arms and name not in args.arms.split(","):
+                continue
+            pages_per_req = -(-(PREFIX_LEN + args.warmup + args.steps + 2) // PAGE_SIZE)
+            engine = _engine_for(cfg, args.batch * pages_per_req + 2 * (PREFILL_TOKENS // PAGE_SIZE) + 8, args.batch + 2)
+            shim = {"vocab_size": vocab}
+            prefill_ms, _ = time_prefill(engine, shim, args.warmup)
+            dec, _ = time_decode(engine, shim, args.batch, args.steps, args.warmup, seed=1)
+            point[name] = {"prefill_tok_s": round(PREFILL_TOKENS / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
+                           "decode_tok_s": round(dec["tok_s"], 1), "decode_ms_per_step": round(dec["ms_per_step"], 4),
+                           "weight_gb": round(engine.model.weight_bytes() / 1e9, 3)}
+            del engine
+            torch.cuda.empty_cache()
+        if not args.no_points:
+            point["kernels"] = tudulix_kernels(pk, size)
+        points.append(point)
+        torch.cuda.empty_cache()
+    clocks.stop()
+    print(json.dumps({"metric": "Tudulix beside Nulilix, Kolisun and Qwen3 dense at equal layer sizes: prefill and decode tokens a second, device-timed",
+                      "unit": "tok/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours", "steps": args.steps,
+                      "warmup": args.warmup, "config": {"batch": args.batch, "prefix_len": PREFIX_LEN, "prefill_tokens": PREFILL_TOKENS,
+                                                        "page_size": PAGE_SIZE, "l2": "inputs_exceed_l2 (steps), flushed (kernels)"},
+                      "points": points, "clocks": clocks.summary([(t_begin, time.time())])}))
+    return 0
+
+
 def serve(args):
     """A mixed continuous batch through ``Engine.generate`` (host tokens in, host tokens out): ``--requests`` prompts
     of uniform random ids with lengths uniform in [128, 2048], prompts cut into portions of ``--prefill-chunk``
@@ -1417,13 +1649,14 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--timeline", action="store_true",
                     help="print the kernels' timeline of one layer of the decode step to stderr (needs PRELUDE_TIMELINE=1 in the environment)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "pabelix", "kolisun", "nedesun", "pepolorn", "nulilix"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "pabelix", "kolisun", "nedesun", "pepolorn", "nulilix", "tudulix"],
                     help="serving: a mixed continuous batch through Engine.generate instead of the decode step (a line of its own); "
                          "pabelix, kolisun: that design beside Qwen3 dense at equal layer sizes (a line of its own); "
                          "nedesun, pepolorn: that design beside Kolisun and Qwen3 dense at equal layer sizes (a line of its own); "
-                         "nulilix: that design beside Pepolorn, Kolisun and Qwen3 dense at equal layer sizes (a line of its own)")
-    ap.add_argument("--sizes", default="2k,4k", help="pabelix, kolisun, nedesun, pepolorn, nulilix: which layer sizes to run (2k, 4k)")
-    ap.add_argument("--arms", default="", help="nulilix: which of the models to run (default: all)")
+                         "nulilix: that design beside Pepolorn, Kolisun and Qwen3 dense at equal layer sizes (a line of its own); "
+                         "tudulix: that design beside Nulilix, Kolisun and Qwen3 dense at equal layer sizes (a line of its own)")
+    ap.add_argument("--sizes", default="2k,4k", help="pabelix, kolisun, nedesun, pepolorn, nulilix, tudulix: which layer sizes to run (2k, 4k)")
+    ap.add_argument("--arms", default="", help="nulilix, tudulix: which of the models to run (default: all)")
     ap.add_argument("--requests", type=int, default=32, help="serving: number of requests")
     ap.add_argument("--prefill-chunk", type=int, default=512, help="serving: tokens per portion of a prompt")
     ap.add_argument("--new-tokens", type=int, default=256, help="serving: generated tokens per request")
@@ -1463,6 +1696,9 @@ def main():
     if args.workload == "nulilix":
         args.layers = 0 if args.layers == MODEL["num_hidden_layers"] else args.layers
         return nulilix_compare(args)
+    if args.workload == "tudulix":
+        args.layers = 0 if args.layers == MODEL["num_hidden_layers"] else args.layers
+        return tudulix_compare(args)
     import torch
     pk = peaks()
     # cache: the largest point (64 requests) with room for prefix + generated tokens, in whole pages
