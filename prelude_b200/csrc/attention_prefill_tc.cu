@@ -393,17 +393,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&p_full[m])) : "memory");
         }
         if (n_m[m] > 0) {
+            const int head = kvh * G + hg;
+            // the row's gates are asked for while its last product runs
+            uint4 gates[T::VD / 8];
+            if (pp.gate_full && valid) {
+                const __nv_bfloat16* src = pp.gate + (size_t)(q_base + tok0 + tl) * pp.ld_gate + (size_t)head * pp.vd;
+#pragma unroll
+                for (int i = 0; i < T::VD / 8; ++i)
+                    if (i * 8 < pp.vd) gates[i] = *reinterpret_cast<const uint4*>(src + i * 8);
+            }
             if (ok) ok = mbar_wait_bounded(&o_full[m], 0);
             if (__all_sync(0xffffffffu, ok)) {
                 tc_fence_after();
-                const int head = kvh * G + hg;
                 if (pp.sink != nullptr && m_ref != -INFINITY) l += ex2_approx(fmaf(pp.sink[head], 1.4426950408889634f, -m_ref));
                 float inv = l > 0.f ? 1.0f / l : 0.f;
                 if (pp.gate != nullptr && valid && !pp.gate_full)
                     inv *= 1.0f / (1.0f + __expf(-__bfloat162float(pp.gate[(size_t)(q_base + tok0 + tl) * pp.ld_gate + head])));
                 __nv_bfloat16* dst = p.out + ((size_t)(q_base + tok0 + (valid ? tl : 0)) * p.n_heads + kvh * G + hg) * pp.vd;
-                const __nv_bfloat16* gates = pp.gate_full ? pp.gate + (size_t)(q_base + tok0 + (valid ? tl : 0)) * pp.ld_gate + (size_t)head * pp.vd : nullptr;
-#pragma unroll 1
+#pragma unroll
                 for (int c = 0; c < T::VD; c += 32) {
                     uint32_t orr[32];
                     tc_tmem_ld32(o_addr + c, orr);
@@ -413,14 +420,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                         for (int i = 0; i < 32; i += 8) {
                             if (c + i >= pp.vd) break;
                             uint4 w;
-                            if (gates != nullptr) {
-                                const uint4 raw = *reinterpret_cast<const uint4*>(gates + c + i);
-                                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+                            if (pp.gate_full) {
+                                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&gates[(c + i) / 8]);
 #pragma unroll
                                 for (int u = 0; u < 4; ++u) {
                                     const float2 g = __bfloat1622float2(h[u]);
-                                    orr[i + 2 * u] = __float_as_uint(__uint_as_float(orr[i + 2 * u]) / (1.0f + __expf(-g.x)));
-                                    orr[i + 2 * u + 1] = __float_as_uint(__uint_as_float(orr[i + 2 * u + 1]) / (1.0f + __expf(-g.y)));
+                                    orr[i + 2 * u] = __float_as_uint(__fdividef(__uint_as_float(orr[i + 2 * u]), 1.0f + __expf(-g.x)));
+                                    orr[i + 2 * u + 1] = __float_as_uint(__fdividef(__uint_as_float(orr[i + 2 * u + 1]), 1.0f + __expf(-g.y)));
                                 }
                             }
                             w.x = pack_bf16(__uint_as_float(orr[i]) * inv, __uint_as_float(orr[i + 1]) * inv);

@@ -1296,16 +1296,21 @@ __device__ __forceinline__ float moe_block_sum(float v, float* red) {
     return total;
 }
 
-template <typename TY, typename TS, typename TO, int V, int IT>
-__global__ void __launch_bounds__(256) moe_sum_normed_kernel(const TY* __restrict__ y, const TS* __restrict__ shared, TO* __restrict__ out, MoeSumNormArgs a) {
+// AHEAD (a few tokens): both scales, written by no kernel, are asked for before the wait; else (a prompt step) they come from
+// the cache when they are needed, which leaves registers for two blocks on a multiprocessor.
+template <typename TY, typename TS, typename TO, int V, int IT, bool AHEAD>
+__global__ void __launch_bounds__(512, AHEAD ? 1 : 2) moe_sum_normed_kernel(const TY* __restrict__ y, const TS* __restrict__ shared, TO* __restrict__ out,
+                                                                            MoeSumNormArgs a) {
     pb_grid_dep_launch();
-    __shared__ float red[2][8];
+    __shared__ float red[2][16];
     const int i = blockIdx.x;
     float gv[IT][V], g[IT][V];
+    if constexpr (AHEAD) {
 #pragma unroll
-    for (int it = 0; it < IT; ++it) {                        // written by no kernel: before the wait
-        const int col = (it * blockDim.x + threadIdx.x) * V;
-        if (col < a.width) { moe_ldv<V>(a.gain_v + col, gv[it]); moe_ldv<V>(a.gain + col, g[it]); }
+        for (int it = 0; it < IT; ++it) {
+            const int col = (it * blockDim.x + threadIdx.x) * V;
+            if (col < a.width) { moe_ldv<V>(a.gain_v + col, gv[it]); moe_ldv<V>(a.gain + col, g[it]); }
+        }
     }
     pb_grid_dep_wait();
     const int t = a.rows ? a.rows[i] : i;
@@ -1361,6 +1366,7 @@ __global__ void __launch_bounds__(256) moe_sum_normed_kernel(const TY* __restric
     for (int it = 0; it < IT; ++it) {
         const int col = (it * blockDim.x + threadIdx.x) * V;
         if (col >= a.width) continue;
+        if constexpr (!AHEAD) moe_ldv<V>(a.gain_v + col, gv[it]);
 #pragma unroll
         for (int e = 0; e < V; ++e) r[it][e] += v[it][e] * inv_v * gv[it][e];
         if (a.plus) {
@@ -1378,6 +1384,7 @@ __global__ void __launch_bounds__(256) moe_sum_normed_kernel(const TY* __restric
     for (int it = 0; it < IT; ++it) {
         const int col = (it * blockDim.x + threadIdx.x) * V;
         if (col >= a.width) continue;
+        if constexpr (!AHEAD) moe_ldv<V>(a.gain + col, g[it]);
         float o[V];
 #pragma unroll
         for (int e = 0; e < V; ++e) o[e] = r[it][e] * inv * g[it][e];
@@ -1388,7 +1395,7 @@ __global__ void __launch_bounds__(256) moe_sum_normed_kernel(const TY* __restric
 // Whether pb_moe_sum_normed takes rows of `width`: multiples of the elements of 16 bytes, what a block's registers hold.
 PB_API int pb_moe_sum_normed_supported(int width, int dtype) {
     const int v = dtype == PB_F32 ? 4 : 8;
-    return width > 0 && width % v == 0 && width / v <= 256 * (dtype == PB_F32 ? 8 : 4) ? 1 : 0;
+    return width > 0 && width % v == 0 && width / v <= 512 * (dtype == PB_F32 ? 4 : 2) ? 1 : 0;
 }
 
 // y, shared as for pb_moe_sum; gain_v, gain float32 [width] as applied; res float32 [n_tokens, width]; plus null or of res's
@@ -1409,17 +1416,18 @@ PB_API int pb_moe_sum_normed(const void* y, int y_dtype, const int32_t* place_of
     if (n_out == 0) return 0;
     const int pieces = width / V;
     int threads = 32;
-    while (threads < 256 && threads < pieces) threads <<= 1;
+    while (threads < 512 && threads < pieces) threads <<= 1;
     const int its = (pieces + threads - 1) / threads;
     const MoeSumNormArgs a{place_of, weights, shared_parts, (size_t)shared_stride, gain_v, gain, plus, res, rows, eps_v, eps, n_tokens, top, width};
-#define MOE_SUM_AT(TY, TS, TO, VV, IT) \
-    pb_launch(moe_sum_normed_kernel<TY, TS, TO, VV, IT>, dim3(n_out), dim3(threads), 0, stream, (const TY*)y, (const TS*)shared, (TO*)out, a)
+    const bool few = n_out <= 148;
+#define MOE_SUM_AT(TY, TS, TO, VV, IT)                                                                                                \
+    pb_launch(few ? moe_sum_normed_kernel<TY, TS, TO, VV, IT, true> : moe_sum_normed_kernel<TY, TS, TO, VV, IT, false>, dim3(n_out), dim3(threads), 0, \
+              stream, (const TY*)y, (const TS*)shared, (TO*)out, a)
 #define MOE_SUM(TY, TS, TO, VV)                                  \
     do {                                                         \
         if (its <= 1) MOE_SUM_AT(TY, TS, TO, VV, 1);             \
         else if (its <= 2) MOE_SUM_AT(TY, TS, TO, VV, 2);        \
-        else if (its <= 4) MOE_SUM_AT(TY, TS, TO, VV, 4);        \
-        else MOE_SUM_AT(TY, TS, TO, VV, 8);                      \
+        else MOE_SUM_AT(TY, TS, TO, VV, (VV == 4 ? 4 : 2));      \
     } while (0)
     if (dtype == PB_F32) MOE_SUM(float, float, float, 4);
     else if (dtype == PB_BF16) {
