@@ -265,8 +265,8 @@ def test_latent_attention_over_a_window_with_a_gate_per_element_equals_the_plain
 
 
 @BOTH
-@pytest.mark.parametrize("kind,window,page", [("attention", 72, 16), ("attention", 128, 16), ("attention", 33, 8), ("attention", 200, 64),
-                                              ("latent_attention", 72, 16), ("latent_attention", 128, 16), ("latent_attention", 33, 8),
+@pytest.mark.parametrize("kind,window,page", [("attention", 75, 16), ("attention", 128, 16), ("attention", 33, 8), ("attention", 200, 64),
+                                              ("latent_attention", 75, 16), ("latent_attention", 128, 16), ("latent_attention", 33, 8),
                                               ("latent_attention", 200, 64)])
 def test_a_key_is_seen_until_it_leaves_the_window(dtype, kind, window, page):
     """One early token's key stands out by so much that every query that sees it sees nothing else: the last position that
@@ -406,7 +406,7 @@ def test_router_chooses_by_biased_logits_and_weighs_the_chosen_alone(experts, to
 @pytest.mark.parametrize("experts,top,ff,limit,shared,T,width", [
     (6, 2, 10, 0.8, (14, 0.4), 37, 48), (5, 3, 14, 1.5, None, 1, 48), (8, 4, 64, 0.7, (96, 1.2), 300, 64), (2, 1, 16, 1.0, (16, 1.0), 9, 48),
     (16, 2, 32, 2.0, (64, 0.5), 70, 128), (2, 2, 64, 0.6, (128, 0.9), 400, 64), (4, 2, 128, 1.1, (256, 0.7), 900, 128), (32, 4, 64, 0.9, (64, 2.0), 8, 256),
-    (3, 1, 7, 0.5, (5, 0.8), 6, 33), (4, 1, 24, 1.0, (8, 0.3), 50, 40), (1, 1, 96, 1.3, (48, 0.9), 800, 64), (12, 2, 96, 2.0, (128, 1.0), 16, 96)])
+    (3, 1, 7, 0.5, (5, 0.8), 6, 33), (4, 1, 24, 1.0, (8, 0.3), 50, 40), (1, 1, 96, 1.3, (48, 0.9), 800, 64), (14, 3, 88, 1.7, (112, 1.2), 16, 96)])
 def test_experts_with_the_clamped_unit_equal_the_plain_ones(dtype, experts, top, ff, limit, shared, T, width):
     """A decode step's few tokens, prompt steps on every tile height, and steps long enough for the paired-block kernel; many
     gate and up sums lie beyond the limits, on both sides, and the shared expert has a limit of its own."""
